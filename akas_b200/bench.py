@@ -358,10 +358,10 @@ def bench_experts(tokens: int, c: int, f: int, experts: int = 14, identity: int 
         st = ops._stream
         p = lambda t: t.data_ptr()
         sort = lambda: ops._fn("moe_grouped", "akas_moe_sort")(p(h), c, p(chosen), p(row_of_pair), p(tile_expert), p(plan), p(srt),
-                                                              tokens, top, c, experts, st())
+                                                              tokens, top, c, experts, None, st())
         gemm = ops._fn("moe_grouped", "akas_moe_grouped_gemm")
-        up = lambda: gemm(p(srt), p(w_gate_up), p(act), p(tile_expert), p(plan), cap, experts, 2 * f, c, 2, st())
-        down = lambda: gemm(p(act), p(w_down), p(y), p(tile_expert), p(plan), cap, experts, c, f, 1, st())
+        up = lambda: gemm(p(srt), p(w_gate_up), p(act), p(tile_expert), p(plan), cap, experts, 2 * f, c, 2, 0, st())
+        down = lambda: gemm(p(act), p(w_down), p(y), p(tile_expert), p(plan), cap, experts, c, f, 1, 0, st())
         comb = lambda: ops._fn("moe_grouped", "akas_moe_combine")(p(h), c, p(y), p(row_of_pair), p(weights), p(out), tokens, top, c, None, None, None, None, 0.0, st())
         sort()
         for name, fn, work in (("sort_ms", sort, 0.0), ("gate_up_ms", up, 2.0 * real * 2 * c * f), ("down_ms", down, 2.0 * real * c * f),

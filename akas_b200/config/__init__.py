@@ -9,6 +9,8 @@ from .kidarax import ARCHITECTURE as KIDARAX_ARCHITECTURE
 from .kidarax import KidaraxConfig
 from .lfm2 import ARCHITECTURE as LFM2_ARCHITECTURE
 from .lfm2 import ConfigError, Lfm2Config
+from .pekodra import ARCHITECTURE as PEKODRA_ARCHITECTURE
+from .pekodra import PekodraConfig
 from .penopel import ARCHITECTURE as PENOPEL_ARCHITECTURE
 from .penopel import PenopelConfig
 from .registry import (
@@ -45,9 +47,10 @@ register_architecture(GIGUSUN_ARCHITECTURE, GigusunConfig)
 register_architecture(GIRELIX_ARCHITECTURE, GirelixConfig)
 register_architecture(PENOPEL_ARCHITECTURE, PenopelConfig)
 register_architecture(KIDARAX_ARCHITECTURE, KidaraxConfig)
+register_architecture(PEKODRA_ARCHITECTURE, PekodraConfig)
 
 __all__ = [
-    "AttentionSpec", "ConfigError", "DecayedLinearAttentionSpec", "DynamicTanhSpec", "GatedMLPSpec", "LatentAttentionSpec", "PenopelConfig", "GirelixConfig", "KidaraxConfig", "MLPSpec", "ParallelMixerSpec", "RoutedExpertsSpec", "EngineConfig", "GatedDeltaSpec", "GatedLinearAttentionSpec", "GigusunConfig", "LayerSpec",
+    "AttentionSpec", "ConfigError", "DecayedLinearAttentionSpec", "DynamicTanhSpec", "GatedMLPSpec", "LatentAttentionSpec", "PekodraConfig", "PenopelConfig", "GirelixConfig", "KidaraxConfig", "MLPSpec", "ParallelMixerSpec", "RoutedExpertsSpec", "EngineConfig", "GatedDeltaSpec", "GatedLinearAttentionSpec", "GigusunConfig", "LayerSpec",
     "Lfm2Config", "ModelSpec", "PartSpec", "PolyNormMLPSpec",
     "RMSNormSpec", "RopeSpec", "ScheduleEntry", "ShortConvSpec", "SwiGLUSpec", "architecture_of",
     "architectures", "config_from_dict", "load_config", "register_architecture",

@@ -106,6 +106,9 @@ class AttentionSpec:
     # False: the layer has no key and value projections; it reads the cache of another layer (the run order names
     # whose), which holds that layer's keys after their rotation and its values, with queries and a mask of its own.
     own_kv: bool = True
+    # A number: after the position encoding every head of q and k is divided by sqrt(mean(x^2) + this number) over the
+    # whole head, without a weight (where ``qk_norm`` is a norm with a weight in front of the position encoding). None: not.
+    qk_unit_eps: Optional[float] = None
 
     @property
     def value_dim(self) -> int:
@@ -116,7 +119,7 @@ class AttentionSpec:
         """Whether the layer needs what only the general attention kernels compute."""
         return bool(self.v_head_dim not in (None, self.head_dim) or self.softcap or self.distance_bias or self.keep_first
                     or self.sink or self.gate or self.values_are_keys or getattr(self.position, "interleaved", False)
-                    or self.bias or not self.own_kv)
+                    or self.bias or not self.own_kv or self.qk_unit_eps is not None)
 
 
 @dataclass(frozen=True)
@@ -267,7 +270,9 @@ class RoutedExpertsSpec:
     scores as they are; ``weight_on="input"``: the weight multiplies the expert's input, the result is
     sum expert(w x), where otherwise it is sum w expert(x); ``shared_size`` F_s: one more expert of that hidden size
     (tensors ``shared.{gate,up,down}``) that every token passes, added to the sum, and with ``shared_gate`` times
-    sigmoid(W_sg x), one number per token (``shared.sg`` [1, hidden])."""
+    sigmoid(W_sg x), one number per token (``shared.sg`` [1, hidden]); ``gated`` False: the experts and the
+    shared one have no gate matrix (tensors ``up`` and ``down`` alone) and compute W_down act(W_up x) with ``activation``
+    one of "relu2" (the square of max(z, 0)), "gelu_tanh", "silu"."""
 
     hidden_size: int
     intermediate_size: int
@@ -282,6 +287,8 @@ class RoutedExpertsSpec:
     weight_on: str = "output"
     shared_size: Optional[int] = None
     shared_gate: bool = False
+    gated: bool = True
+    activation: str = "silu"
     kind: str = "routed_experts"
     names: Mapping[str, str] = field(default_factory=dict)
 
@@ -344,7 +351,8 @@ class LayerSpec:
     mixer_post_norm_name: Optional[str] = None
     ffn_post_norm_name: Optional[str] = None
     # What the "parallel" arrangement adds: h += residual_multiplier * (mixer_scale * mixer(n) + ffn_scale * ffn(n))
-    # with ONE norm n = mixer_norm(h) that both sublayers read; the two scales are tensors [hidden] (None: ones).
+    # with ONE norm n = mixer_norm(h) that both sublayers read, or, where ``ffn_norm`` is given, a norm for each, both of
+    # the same h; the two scales are tensors [hidden] (None: ones).
     residual_multiplier: float = 1.0
     mixer_scale_name: Optional[str] = None
     ffn_scale_name: Optional[str] = None
@@ -359,12 +367,14 @@ class ScheduleEntry:
     entry's index reads that entry's cache and writes nothing into it (the mixer
     is told ``write=False``). Naming a layer in two entries runs its weights twice,
     each time with the cache of its own entry. ``add_embedding``: before the layer runs, the embedding's output (the
-    stream as it was in front of the first entry) is added to the stream once more.
+    stream as it was in front of the first entry) is added to the stream once more. ``join`` names a tensor
+    W [hidden, 2 hidden]: before the layer runs, the stream x becomes W [x; embedding's output].
     """
 
     layer: int
     cache: Optional[int] = None
     add_embedding: bool = False
+    join: Optional[str] = None
 
 
 @dataclass(frozen=True)

@@ -26,6 +26,8 @@ constexpr int kMaxGroup = 16;  // query heads of a key/value head that one block
 // (page, offset). v may be the very rows of k: the values are then the keys as projected, before the rotation.
 // Where biases are given (float32, one per channel of q, k, v), they are added first, in float32; q, k and v may then
 // be the float32 result of a product (TI) while the pages hold T, so product plus bias is rounded once.
+// unit: there is no norm in front of the rotation; behind it every head of q and k is divided by
+// sqrt(mean of its D squares + eps), without a weight.
 template <typename TI, typename T>
 __global__ void qk_norm_store_kernel(const TI* __restrict__ q, long long ldq, const TI* __restrict__ k, long long ldk,
                                      const TI* __restrict__ v, long long ldv, const float* __restrict__ qw,
@@ -35,7 +37,7 @@ __global__ void qk_norm_store_kernel(const TI* __restrict__ q, long long ldq, co
                                      const int* __restrict__ positions, int page_size, int H, int G, int D, int V, int write,
                                      const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot,
                                      int interleaved, const float* __restrict__ qb, const float* __restrict__ kb,
-                                     const float* __restrict__ vb) {
+                                     const float* __restrict__ vb, int unit) {
   const int n = blockIdx.x;
   const int req = seq_of_token[n];
   if (req < 0) return;
@@ -51,7 +53,19 @@ __global__ void qk_norm_store_kernel(const TI* __restrict__ q, long long ldq, co
     const float* bias = is_q ? (qb != nullptr ? qb + (size_t)head * D : nullptr) : (kb != nullptr ? kb + (size_t)(head - H) * D : nullptr);
     auto at = [&](int d) { return bias != nullptr ? to_f32(src[d]) + bias[d] : to_f32(src[d]); };
     float inv = 1.f;
-    if (w != nullptr) {
+    if (unit) {
+      // the squares of the rotated channels as the rotation leaves them (its tables may carry an amplitude)
+      float ss = 0.f;
+      const int turned = cos_t != nullptr ? rot : 0, half = turned / 2;
+      for (int i = lane; i < half; i += 32) {
+        const float u = at(interleaved ? 2 * i : i), x = at(interleaved ? 2 * i + 1 : i + half);
+        const float c = cos_t[(size_t)n * half + i], sn = sin_t[(size_t)n * half + i];
+        const float ru = fmaf(u, c, -x * sn), rx = fmaf(x, c, u * sn);
+        ss = fmaf(ru, ru, fmaf(rx, rx, ss));
+      }
+      for (int d = turned + lane; d < D; d += 32) { const float x = at(d); ss = fmaf(x, x, ss); }
+      inv = 1.f / sqrtf(warp_sum(ss) / (float)D + eps);
+    } else if (w != nullptr) {
       float ss = 0.f;
       for (int d = lane; d < D; d += 32) { const float x = at(d); ss = fmaf(x, x, ss); }
       ss = warp_sum(ss);
@@ -60,7 +74,7 @@ __global__ void qk_norm_store_kernel(const TI* __restrict__ q, long long ldq, co
     T* dst = is_q ? q_out + ((size_t)n * H + head) * D
                   : k_pool + (((size_t)page * G + (head - H)) * page_size + off) * D;
     if (cos_t == nullptr) {
-      for (int d = lane; d < D; d += 32) dst[d] = from_f32<T>(w != nullptr ? at(d) * inv * w[d] : at(d));
+      for (int d = lane; d < D; d += 32) dst[d] = from_f32<T>(w != nullptr ? at(d) * inv * w[d] : unit ? at(d) * inv : at(d));
       continue;
     }
     const int half = rot / 2;
@@ -69,10 +83,11 @@ __global__ void qk_norm_store_kernel(const TI* __restrict__ q, long long ldq, co
       float u = at(a), x = at(b);
       if (w != nullptr) { u *= inv * w[a]; x *= inv * w[b]; }
       const float c = cos_t[(size_t)n * half + i], sn = sin_t[(size_t)n * half + i];
-      dst[a] = from_f32<T>(fmaf(u, c, -x * sn));
-      dst[b] = from_f32<T>(fmaf(x, c, u * sn));
+      const float ru = fmaf(u, c, -x * sn), rx = fmaf(x, c, u * sn);
+      dst[a] = from_f32<T>(unit ? ru * inv : ru);
+      dst[b] = from_f32<T>(unit ? rx * inv : rx);
     }
-    for (int d = rot + lane; d < D; d += 32) dst[d] = from_f32<T>(w != nullptr ? at(d) * inv * w[d] : at(d));
+    for (int d = rot + lane; d < D; d += 32) dst[d] = from_f32<T>(w != nullptr ? at(d) * inv * w[d] : unit ? at(d) * inv : at(d));
   }
   if (write) {
     for (int i = threadIdx.x; i < G * V; i += blockDim.x) {
@@ -264,21 +279,22 @@ AKAS_API int akas_qk_norm_store(const void* q, long long ldq, const void* k, lon
                                 const int* block_table, int max_blocks, const int* seq_of_token, const int* positions,
                                 int page_size, int N, int H, int G, int D, int V, int write, int dtype, const float* cos_t,
                                 const float* sin_t, int rot, int interleaved, int in_dtype, const float* qb, const float* kb,
-                                const float* vb, cudaStream_t stream) {
+                                const float* vb, int unit, cudaStream_t stream) {
   if (N <= 0) return 0;
+  if (unit && (qw != nullptr || kw != nullptr)) return (int)cudaErrorInvalidValue;
   if (cos_t != nullptr && (rot <= 0 || rot % 2 || rot > D)) return (int)cudaErrorInvalidValue;
   if (dtype == AKAS_F32 && in_dtype != AKAS_F32) return (int)cudaErrorInvalidValue;
   if (dtype == AKAS_F32)
     return launch_ordinary(qk_norm_store_kernel<float, float>, dim3(N), dim3(128), 0, stream, (const float*)q, ldq, (const float*)k, ldk,
                           (const float*)v, ldv, qw, kw, eps, (float*)q_out, (float*)k_pool, (float*)v_pool, block_table,
-                          max_blocks, seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb);
+                          max_blocks, seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb, unit);
   if (in_dtype == AKAS_F32)
     return launch_ordinary(qk_norm_store_kernel<float, bf16>, dim3(N), dim3(128), 0, stream, (const float*)q, ldq, (const float*)k, ldk,
                           (const float*)v, ldv, qw, kw, eps, (bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool, block_table, max_blocks,
-                          seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb);
+                          seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb, unit);
   return launch_ordinary(qk_norm_store_kernel<bf16, bf16>, dim3(N), dim3(128), 0, stream, (const bf16*)q, ldq, (const bf16*)k, ldk,
                         (const bf16*)v, ldv, qw, kw, eps, (bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool, block_table, max_blocks,
-                        seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb);
+                        seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb, unit);
 }
 
 template <typename T, typename TG>

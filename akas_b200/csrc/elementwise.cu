@@ -298,6 +298,115 @@ AKAS_API int akas_scaled_add(float* x, const float* a, const float* ls_a, const 
                          mult, total, C, vec);
 }
 
+// Two RMSNorms of the same float32 row with weights of their own: the row is read once and stays in registers between
+// the sum of squares and the two scalings (groups of 8 elements; PER_THREAD of them a thread). One block per row.
+template <typename TO, int PER_THREAD>
+__global__ void __launch_bounds__(256)
+rmsnorm_pair_rows_kernel(const float* __restrict__ x, const float* __restrict__ w1, const float* __restrict__ w2,
+                         TO* __restrict__ y1, TO* __restrict__ y2, int C, float eps, int zero_centered) {
+  __shared__ float scratch[32];
+  const float* src = x + (size_t)blockIdx.x * C;
+  const float shift = zero_centered ? 1.f : 0.f;
+  float v[PER_THREAD][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int p = 0; p < PER_THREAD; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * 8;
+    if (c < C) {
+      load8(src + c, v[p]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss = fmaf(v[p][e], v[p][e], ss);
+    }
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.f / sqrtf(ss / (float)C + eps);
+#pragma unroll
+  for (int p = 0; p < PER_THREAD; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * 8;
+    if (c < C) {
+      float g[8], o[8];
+      load8(w1 + c, g);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) o[e] = v[p][e] * inv * (g[e] + shift);
+      store8(y1 + (size_t)blockIdx.x * C + c, o);
+      load8(w2 + c, g);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) o[e] = v[p][e] * inv * (g[e] + shift);
+      store8(y2 + (size_t)blockIdx.x * C + c, o);
+    }
+  }
+}
+
+// The same for rows of any width.
+template <typename TO>
+__global__ void rmsnorm_pair_kernel(const float* __restrict__ x, const float* __restrict__ w1, const float* __restrict__ w2,
+                                    TO* __restrict__ y1, TO* __restrict__ y2, int C, float eps, int zero_centered) {
+  __shared__ float scratch[32];
+  const float* src = x + (size_t)blockIdx.x * C;
+  const float shift = zero_centered ? 1.f : 0.f;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < C; c += blockDim.x) ss = fmaf(src[c], src[c], ss);
+  ss = block_sum(ss, scratch);
+  const float inv = 1.f / sqrtf(ss / (float)C + eps);
+  for (int c = threadIdx.x; c < C; c += blockDim.x) {
+    const float n = src[c] * inv;
+    y1[(size_t)blockIdx.x * C + c] = from_f32<TO>(n * (w1[c] + shift));
+    y2[(size_t)blockIdx.x * C + c] = from_f32<TO>(n * (w2[c] + shift));
+  }
+}
+
+template <typename TO>
+static int launch_rmsnorm_pair(const float* x, const float* w1, const float* w2, TO* y1, TO* y2, int M, int C, float eps,
+                               int zero_centered, cudaStream_t stream) {
+  const bool aligned = ((uintptr_t)x | (uintptr_t)w1 | (uintptr_t)w2 | (uintptr_t)y1 | (uintptr_t)y2) % 16 == 0;
+  if (C % 8 || C > 8192 || !aligned)
+    return launch_ordinary(rmsnorm_pair_kernel<TO>, dim3(M), dim3(C >= 512 ? 256 : 128), 0, stream, x, w1, w2, y1, y2, C, eps, zero_centered);
+  const dim3 block(C >= 2048 ? 256 : (C / 8 + 31) / 32 * 32);
+#define AKAS_PAIR(P) return launch_ordinary(rmsnorm_pair_rows_kernel<TO, P>, dim3(M), block, 0, stream, x, w1, w2, y1, y2, C, eps, zero_centered)
+  if (C <= 2048) AKAS_PAIR(1);
+  if (C <= 4096) AKAS_PAIR(2);
+  AKAS_PAIR(4);
+#undef AKAS_PAIR
+}
+
+AKAS_API int akas_rmsnorm_pair(const float* x, const float* w1, const float* w2, void* y1, void* y2, int M, int C, float eps,
+                               int zero_centered, int out_dtype, cudaStream_t stream) {
+  if (M <= 0) return 0;
+  if (out_dtype == AKAS_F32) return launch_rmsnorm_pair(x, w1, w2, (float*)y1, (float*)y2, M, C, eps, zero_centered, stream);
+  return launch_rmsnorm_pair(x, w1, w2, (bf16*)y1, (bf16*)y2, M, C, eps, zero_centered, stream);
+}
+
+// out[n, 0..C) = x[n, 0..C) rounded to the output's type; the output's rows have a pitch of their own (ldo elements), so
+// they may be a part of wider rows. VEC: 8 elements move at a time.
+template <typename TO, bool VEC>
+__global__ void round_rows_kernel(const float* __restrict__ x, TO* __restrict__ out, long long ldo, long long items, int per_row) {
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= items) return;
+  const long long n = i / per_row;
+  const int c = (int)(i % per_row);
+  if (VEC) {
+    float v[8];
+    load8(x + i * 8, v);
+    store8(out + n * ldo + c * 8, v);
+  } else {
+    out[n * ldo + c] = from_f32<TO>(x[i]);
+  }
+}
+
+AKAS_API int akas_round_rows(const float* x, void* out, long long ldo, int N, int C, int out_dtype, cudaStream_t stream) {
+  if (N <= 0 || C <= 0) return 0;
+  if (ldo < C) return (int)cudaErrorInvalidValue;
+  const bool vec = C % 8 == 0 && ldo % 8 == 0 && ((uintptr_t)x | (uintptr_t)out) % 16 == 0;
+  const int per_row = vec ? C / 8 : C;
+  const long long items = (long long)N * per_row;
+  const dim3 grid((unsigned)((items + 255) / 256));
+  if (out_dtype == AKAS_F32)
+    return vec ? launch_ordinary(round_rows_kernel<float, true>, grid, dim3(256), 0, stream, x, (float*)out, ldo, items, per_row)
+               : launch_ordinary(round_rows_kernel<float, false>, grid, dim3(256), 0, stream, x, (float*)out, ldo, items, per_row);
+  return vec ? launch_ordinary(round_rows_kernel<bf16, true>, grid, dim3(256), 0, stream, x, (bf16*)out, ldo, items, per_row)
+             : launch_ordinary(round_rows_kernel<bf16, false>, grid, dim3(256), 0, stream, x, (bf16*)out, ldo, items, per_row);
+}
+
 // PolyNorm of rows: out = a N(z) + b N(z^2) + c N(z^3) + e with N(x) = x / sqrt(mean(x^2) + eps) over the row and
 // the powers taken element by element; coeffs = (a, b, c, e). One block per row; powers and sums are float32. VEC: the
 // row's width is a multiple of 8 and rows start on 16 bytes, so 8 elements move at a time.

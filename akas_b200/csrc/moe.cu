@@ -8,6 +8,7 @@
 // they have no matrices and return their input. Options: `sigmoid`, s = 1 / (1 + exp(-z)) per output instead of the
 // softmax; no correction (a null pointer); `renorm` 0, the weights are the chosen s as they are; `extra` more rows of
 // W_r behind the R that compete, whose sigmoids are returned beside the choice (gates that read the router's input).
+// Without a correction the choice goes by the logits themselves, which order as the scores do.
 //
 // Experts, token by token (moe_gate_up, moe_down): act[pair] = silu(W_gate h) * (W_up h) for every (token, chosen
 // real expert) pair, then out[n] = sum over the token's chosen outputs of weight * (W_down act, or h for an identity
@@ -15,7 +16,8 @@
 // a token's result does not depend on what else the step holds. Weights of all experts are stacked: gate and up as
 // [experts, 2 F, C] (gate rows first), down as [experts, C, F]. Where the weight multiplies the expert's INPUT
 // (out[n] = sum expert(w h)), moe_gate_up gets the weights and scales both of its float32 sums (W (w h) = w (W h))
-// before the activation, and moe_down gets none. moe_down can also add a dense result of every token (a shared
+// before the activation, and moe_down gets none. Ungated experts (`plain`, an AKAS_PLAIN_* activation): the stack is
+// [experts, F, C] and act[pair] = act(W_up h). moe_down can also add a dense result of every token (a shared
 // expert's), times a gate per token.
 #include "common.cuh"
 
@@ -28,6 +30,12 @@ constexpr int kRouteChunk = 2048; // channels of h staged at a time (64 KB of fl
 constexpr int kRouteOutputs = 4;  // router outputs whose rows a warp reads at the same time
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// An activation without a gate in full float32 (AKAS_PLAIN_*).
+__device__ __forceinline__ float plain_activation(float x, int act) {
+  if (act == AKAS_PLAIN_RELU2) { const float r = fmaxf(x, 0.f); return r * r; }
+  if (act == AKAS_PLAIN_GELU_TANH) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * x * x, x, x)));
+  return act == AKAS_PLAIN_SILU ? silu_f(x) : x;
+}
 
 template <typename T>
 __global__ void __launch_bounds__(kRouteTokens * 32)
@@ -161,6 +169,7 @@ moe_route_kernel(const T* __restrict__ h, long long ldh, const float* __restrict
     top_z = warp_max(top_z);
     float sum = 0.f;
     for (int e = lane; e < R; e += 32) {
+      pt[e] = zt[e];  // without a correction: the choice goes by the logits
       const float p = expf(zt[e] - top_z);
       zt[e] = p;
       sum += p;
@@ -169,7 +178,7 @@ moe_route_kernel(const T* __restrict__ h, long long ldh, const float* __restrict
     const float inv = 1.f / sum;
     for (int e = lane; e < R; e += 32) {
       zt[e] *= inv;
-      pt[e] = zt[e] + (correction != nullptr ? correction[e] : 0.f);
+      if (correction != nullptr) pt[e] = zt[e] + correction[e];
     }
   }
   __syncwarp();
@@ -218,22 +227,41 @@ moe_route_kernel(const T* __restrict__ h, long long ldh, const float* __restrict
 }
 
 // One warp per (pair, hidden channel f): both dots over C, act = silu(gate) * up. Pairs of identity experts do nothing.
-// in_weights (or null): the pair's weight multiplies both sums before the activation.
+// in_weights (or null): the pair's weight multiplies both sums before the activation. plain (AKAS_PLAIN_*): no gate, one
+// dot per hidden channel over rows of a stack [experts, F, C], act = that activation of it.
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_gate_up_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w_gate_up, const int* __restrict__ chosen,
-                   T* __restrict__ act, int pairs, int top, int C, int F, int experts, const float* __restrict__ in_weights) {
+                   T* __restrict__ act, int pairs, int top, int C, int F, int experts, const float* __restrict__ in_weights,
+                   int plain) {
   const int pair = blockIdx.x;
   const int e = chosen[pair];
   if (e >= experts || e < 0) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   const T* x = h + (size_t)(pair / top) * ldh;
-  const T* wg = w_gate_up + (size_t)e * 2 * F * C;
+  const T* wg = w_gate_up + (size_t)e * (plain ? 1 : 2) * F * C;
   const float scale = in_weights != nullptr ? in_weights[pair] : 1.f;
   constexpr int N = Vec<T>::N;
   const bool vec = C % N == 0 && ldh % N == 0 && ((uintptr_t)h % 16) == 0 && ((uintptr_t)w_gate_up % 16) == 0;
   for (int f = blockIdx.y * warps + warp; f < F; f += gridDim.y * warps) {
     const T* g_row = wg + (size_t)f * C;
+    if (plain) {
+      float sum = 0.f;
+      if (vec) {
+        for (int c = lane * N; c < C; c += 32 * N) {
+          float xv[N], gv[N];
+          load_vec(x + c, xv);
+          load_vec(g_row + c, gv);
+#pragma unroll
+          for (int i = 0; i < N; ++i) sum = fmaf(xv[i], gv[i], sum);
+        }
+      } else {
+        for (int c = lane; c < C; c += 32) sum = fmaf(to_f32(x[c]), to_f32(g_row[c]), sum);
+      }
+      sum = warp_sum(sum) * scale;
+      if (lane == 0) act[(size_t)pair * F + f] = from_f32<T>(plain_activation(sum, plain));
+      continue;
+    }
     const T* u_row = wg + (size_t)(F + f) * C;
     float ag = 0.f, au = 0.f;
     if (vec) {
@@ -343,16 +371,17 @@ AKAS_API int akas_moe_route(const void* h, long long ldh, const float* w, const 
 }
 
 AKAS_API int akas_moe_gate_up(const void* h, long long ldh, const void* w_gate_up, const int* chosen, void* act, int N,
-                              int top, int C, int F, int experts, int dtype, const float* in_weights, cudaStream_t stream) {
+                              int top, int C, int F, int experts, int dtype, const float* in_weights, int plain, cudaStream_t stream) {
   if (N <= 0 || top <= 0 || experts <= 0) return 0;
+  if (plain < AKAS_PLAIN_NONE || plain > AKAS_PLAIN_SILU) return (int)cudaErrorInvalidValue;
   const int pairs = N * top;
   // warps enough to fill the GPU when the pairs are few (a row of F per warp), fewer and longer-lived when they are many
   const dim3 grid(pairs, max(1, min((F + 7) / 8, pairs >= 4096 ? 2 : pairs >= 256 ? 16 : 256)));
   if (dtype == AKAS_F32)
     return launch_ordinary(moe_gate_up_kernel<float>, grid, dim3(256), 0, stream, (const float*)h, ldh, (const float*)w_gate_up,
-                           chosen, (float*)act, pairs, top, C, F, experts, in_weights);
+                           chosen, (float*)act, pairs, top, C, F, experts, in_weights, plain);
   return launch_ordinary(moe_gate_up_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16*)h, ldh, (const bf16*)w_gate_up,
-                         chosen, (bf16*)act, pairs, top, C, F, experts, in_weights);
+                         chosen, (bf16*)act, pairs, top, C, F, experts, in_weights, plain);
 }
 
 AKAS_API int akas_moe_down(const void* h, long long ldh, const void* w_down, const int* chosen, const float* weights,

@@ -9,7 +9,8 @@
 //   moe_gather   copies each pair's token row of h into its row of the sorted buffer.
 //   grouped product (the persistent, TMA-fed, tcgen05 kernel of gemm_tcgen05.cu with an expert per tile): B tiles
 //                come from the stacked matrices [experts * rows, K] at the tile's expert;
-//                  SWIGLU: act[row, F] = silu(gate) * up, bfloat16;   F32: y[row, C] = act . W_down^T, float32.
+//                  SWIGLU: act[row, F] = silu(gate) * up, bfloat16;   F32: y[row, C] = act . W_down^T, float32;
+//                  PLAIN: act[row, F] = an activation without a gate (ungated experts, matrices [experts * F, K]), bfloat16.
 //   moe_combine  out[n] = sum_k weight[n, k] * (y[row of pair (n, k)], or h[n] for an identity expert), in the
 //                order of the choice, float32; or, given the residual stream x, x += mult * (ls_a * a + ls_b * that sum).
 // Every output is a sum over the inner size in the tile order of K, whatever the step holds beside the token, so a
@@ -25,7 +26,7 @@ namespace {
 
 constexpr int BM = 128, STAGES = 4;
 constexpr int THREADS = 192;
-enum { EPI_F32 = 1, EPI_SWIGLU = 2 };
+enum { EPI_F32 = 1, EPI_SWIGLU = 2, EPI_PLAIN = 4 };
 
 __device__ int g_grouped_status = 0;  // 0, or which bounded wait ran out last (1 producer, 2 tensor cores, 3 epilogue)
 
@@ -133,7 +134,8 @@ __global__ void moe_combine_kernel(const bf16* __restrict__ h, long long ldh, co
 template <int BN, int EPI>
 __global__ void __launch_bounds__(THREADS)
 grouped_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-               void* __restrict__ y_, const int* __restrict__ tile_expert, const int* __restrict__ plan, int N, int K, int F) {
+               void* __restrict__ y_, const int* __restrict__ tile_expert, const int* __restrict__ plan, int N, int K, int F,
+               int act) {
   // A tile's B rows are those of its expert in the stacked matrix [experts * N, K]; M is what the plan kernel counted.
   // N: channels of the product (for SWIGLU the stacked height 2F); a tile covers BN of them (SWIGLU: BN/2 gate
   // rows f0.. and BN/2 up rows F + f0..).
@@ -246,6 +248,10 @@ grouped_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
 #pragma unroll
           for (int i = 0; i < 16; ++i) v[i] = __fdividef(v[i], 1.f + __expf(-v[i])) * u[i];  // the fast division: IEEE division cost more than the tile's loads
         }
+        if (EPI == EPI_PLAIN) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) v[i] = plain_activation_fast(v[i], act);
+        }
         const int col = n0 + c;
         if (row < M && col < out_cols) {
           if (EPI == EPI_F32) {
@@ -292,7 +298,7 @@ grouped_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
 
 template <int BN, int EPI>
 int launch(const void* x, const void* w, void* y, const int* tile_expert, const int* plan, int rows_cap, int experts, int N,
-           int K, cudaStream_t stream) {
+           int K, int act, cudaStream_t stream) {
   constexpr int smem = STAGES * (BM * BK * 2 + BN * BK * 2) + 1024;
   static int sms_of[64] = {};
   int device = 0;
@@ -312,7 +318,7 @@ int launch(const void* x, const void* w, void* y, const int* tile_expert, const 
   const int out_cols = EPI == EPI_SWIGLU ? F : N, tile_n = EPI == EPI_SWIGLU ? BN / 2 : BN;
   const long long most = (long long)(rows_cap / BM) * ((out_cols + tile_n - 1) / tile_n);
   const int grid = most < sms ? (int)most : sms;
-  grouped_kernel<BN, EPI><<<grid, THREADS, smem, stream>>>(map_x, map_w, y, tile_expert, plan, N, K, F);
+  grouped_kernel<BN, EPI><<<grid, THREADS, smem, stream>>>(map_x, map_w, y, tile_expert, plan, N, K, F, act);
   return launch_status();
 }
 
@@ -338,20 +344,27 @@ AKAS_API int akas_moe_sort(const void* h, long long ldh, const int* chosen, int*
 }
 
 // epilogue 2: x = sorted [rows_cap, K = C], w = [experts, 2F, C] (N = 2F), y = act [rows_cap, F] bfloat16;
-// epilogue 1: x = act [rows_cap, K = F], w = [experts, C, F] (N = C), y float32 [rows_cap, C].
+// epilogue 1: x = act [rows_cap, K = F], w = [experts, C, F] (N = C), y float32 [rows_cap, C];
+// epilogue 4: x = sorted [rows_cap, K = C], w = [experts, F, C] (N = F), y = act(x . w) [rows_cap, F] bfloat16 with `act`
+// an AKAS_PLAIN_* activation.
 AKAS_API int akas_moe_grouped_gemm(const void* x, const void* w, void* y, const int* tile_expert, const int* plan, int rows_cap,
-                                   int experts, int N, int K, int epilogue, cudaStream_t stream) {
+                                   int experts, int N, int K, int epilogue, int act, cudaStream_t stream) {
   if (rows_cap <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8 || rows_cap % BM || (uintptr_t)x % 16 || (uintptr_t)w % 16 || (uintptr_t)y % 16) return (int)cudaErrorInvalidValue;
   if (epilogue == EPI_SWIGLU) {
     if (N % 2 || (N / 2) % 8) return (int)cudaErrorInvalidValue;
-    return launch<256, EPI_SWIGLU>(x, w, y, tile_expert, plan, rows_cap, experts, N, K, stream);
+    return launch<256, EPI_SWIGLU>(x, w, y, tile_expert, plan, rows_cap, experts, N, K, 0, stream);
+  }
+  if (epilogue == EPI_PLAIN) {
+    if (N % 8 || act < AKAS_PLAIN_NONE || act > AKAS_PLAIN_SILU) return (int)cudaErrorInvalidValue;
+    return N <= 128 ? launch<128, EPI_PLAIN>(x, w, y, tile_expert, plan, rows_cap, experts, N, K, act, stream)
+                    : launch<256, EPI_PLAIN>(x, w, y, tile_expert, plan, rows_cap, experts, N, K, act, stream);
   }
   if (epilogue != EPI_F32) return (int)cudaErrorInvalidValue;
   // (128 x 128 tiles for steps whose 128 x 256 tiles would leave SMs without one were measured and dropped: the down
   // product of 64 tokens over 14 experts took 48 us against 43 us)
-  return N <= 128 ? launch<128, EPI_F32>(x, w, y, tile_expert, plan, rows_cap, experts, N, K, stream)
-                  : launch<256, EPI_F32>(x, w, y, tile_expert, plan, rows_cap, experts, N, K, stream);
+  return N <= 128 ? launch<128, EPI_F32>(x, w, y, tile_expert, plan, rows_cap, experts, N, K, 0, stream)
+                  : launch<256, EPI_F32>(x, w, y, tile_expert, plan, rows_cap, experts, N, K, 0, stream);
 }
 
 AKAS_API int akas_moe_combine(const void* h, long long ldh, const float* y, const int* row_of_pair, const float* weights,

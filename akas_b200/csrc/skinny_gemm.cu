@@ -826,6 +826,16 @@ AKAS_API int akas_skinny_gemm(const void* x, const int* rows, const float* norm_
   return skinny_dispatch(x, rows, norm_w, eps, zero_centered, W, y, M, O, K, in_mode, out_mode, ConvTail{}, stream);
 }
 
+// RMSNorm on the way in (as in_mode 1 above) in front of the gated read-out with its biases and activation: W is the
+// stacked [2F, K] matrix (O = 2F), y bfloat16 [M, F] = act(gate + b_g) * (up + b_u).
+AKAS_API int akas_skinny_gemm_norm_gated(const void* x, const int* rows, const float* norm_w, float eps, int zero_centered,
+                                         const void* W, void* y, int M, int O, int K, const float* bias, int act,
+                                         cudaStream_t stream) {
+  if (act != AKAS_ACT_SILU && act != AKAS_ACT_GELU_TANH) return (int)cudaErrorInvalidValue;
+  const ConvTail tail{nullptr, bias, nullptr, nullptr, nullptr, act, 0, nullptr, nullptr};
+  return skinny_dispatch(x, rows, norm_w, eps, zero_centered, W, y, M, O, K, IN_NORM, OUT_SWIGLU, tail, stream);
+}
+
 // The same with more: in_mode 2, the input rows through a norm without sums, bf16(tanh(alpha x) * norm_w + shift), in
 // front of out modes 0, 1 and 3; a float32 bias on the float32 read-outs (one number per output channel: y = product +
 // bias, or += for the accumulating one) or on the gated read-out ([2F], with `act` 0 silu or 1 the tanh form of gelu:

@@ -3,7 +3,8 @@
 Embedding (times ``ModelSpec.embedding_multiplier`` if the architecture has one, plus a learned position vector
 and through a norm if it has those), the blocks of
 ``ModelSpec.layers`` in the order of ``ModelSpec.schedule`` (a list that may name a layer twice, let an
-entry read another entry's cache, or have the embedding's output added again in front of an entry), the final norm on the rows whose logits are wanted, the head, and the
+entry read another entry's cache, or have the embedding's output added again or joined to the stream by a matrix in
+front of an entry), the final norm on the rows whose logits are wanted, the head, and the
 architecture's ``logit_scale`` and ``logit_softcap`` if it has them. The head is the checkpoint's
 head tensor when it has one, else the embedding:
 src/akas/models/lfm2/weights.py:399-402 and _composition.py:363-380 in kreasof-ai/akas).
@@ -46,6 +47,7 @@ class Decoder:
         self.embedding = None
         self.positions = None  # learned absolute positions [max_context, hidden], where the architecture has them
         self.head = None
+        self.joins: Dict[str, Optional[torch.Tensor]] = {e.join: None for e in self.schedule if getattr(e, "join", None)}
 
     # ------------------------------------------------------------------ weights
 
@@ -59,6 +61,8 @@ class Decoder:
             out[s.position_table_name] = Param((s.max_context, s.hidden_size))
         if self.embedding_norm is not None:
             out.update(norm_params(self.embedding_norm, s.embedding_norm_name))
+        for name in self.joins:
+            out[name] = Param((s.hidden_size, 2 * s.hidden_size))
         for block in self.blocks:
             out.update(block.params())
         return out
@@ -72,6 +76,8 @@ class Decoder:
         if self.embedding_norm is not None:
             load_norm(self.embedding_norm, s.embedding_norm_name, get)
         self.head = get(s.head_name) if s.head_name is not None and has(s.head_name) else self.embedding
+        for name in self.joins:
+            self.joins[name] = get(name)
         for block in self.blocks:
             block.load(get)
 
@@ -109,6 +115,12 @@ class Decoder:
             if chained:
                 ops.chain_flush()
             first = h.clone()
+        # entries that join it to the stream read both side by side, in the compute dtype: the embedding's half is
+        # written once, the stream's half in front of every such entry
+        joined = None
+        if self.joins:
+            joined = torch.empty((h.shape[0], 2 * spec.hidden_size), dtype=self.rt.dtype, device=h.device)
+            ops.round_rows(h, joined[:, spec.hidden_size :])
         for i, entry in enumerate(self.schedule):
             owner = i if entry.cache is None else entry.cache
             block = self.blocks[entry.layer]
@@ -116,6 +128,9 @@ class Decoder:
                 ops.chain_flush()
             if entry.add_embedding:
                 h = ops.scaled_add(h, first, None, None, None, 1.0)
+            if joined is not None and entry.join is not None:
+                ops.round_rows(h, joined[:, : spec.hidden_size])
+                h = ops.linear(joined, self.joins[entry.join], out_dtype=torch.float32)
             h = block.forward(h, ctx, caches[owner], write=entry.cache is None)
         if chained and not getattr(self.final_norm, "chain_safe", False):
             ops.chain_flush()

@@ -31,6 +31,8 @@ _SIGNATURES = {
     "elementwise": {
         "akas_embedding": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "akas_rmsnorm": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p],
+        "akas_rmsnorm_pair": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_void_p],
+        "akas_round_rows": [c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p],
         "akas_swiglu": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "akas_take_tokens": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "akas_zero_row": [c_void_p, c_longlong, c_int, c_int, c_longlong, c_void_p],
@@ -55,7 +57,7 @@ _SIGNATURES = {
         "akas_moe_route": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                            c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "akas_moe_gate_up": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                             c_void_p, c_void_p],
+                             c_void_p, c_int, c_void_p],
         "akas_moe_down": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                           c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_longlong,
                           c_void_p],
@@ -84,7 +86,7 @@ _SIGNATURES = {
         "akas_qk_norm_store": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_float,
                                c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p,
-                               c_void_p, c_void_p],
+                               c_void_p, c_int, c_void_p],
         "akas_attention_general": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int,
                                    c_int, c_float, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_int,
                                    c_int, c_int, c_int, c_void_p, c_float, c_longlong, c_longlong, c_int, c_int, c_void_p],
@@ -101,7 +103,8 @@ _SIGNATURES = {
         "akas_moe_grouped_takes": [c_int, c_int, c_int],
         "akas_moe_sort": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                           c_void_p, c_void_p],
-        "akas_moe_grouped_gemm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "akas_moe_grouped_gemm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                                  c_void_p],
         "akas_moe_combine": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p,
                              c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_longlong, c_void_p],
         "akas_moe_grouped_status": [],
@@ -180,6 +183,8 @@ _SIGNATURES = {
                                   c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "akas_skinny_gemm_more": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                   c_int, c_int, c_void_p, c_int, c_void_p],
+        "akas_skinny_gemm_norm_gated": [c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+                                        c_void_p, c_int, c_void_p],
         "akas_skinny_gemm_status": [],
     },
     "decode_chain": {
@@ -452,6 +457,33 @@ def rmsnorm(x, weight, eps, zero_centered, out_dtype, rows=None):
     _check(_fn("elementwise", "akas_rmsnorm")(_ptr(x), _ptr(weight), _ptr(out), _ptr(rows), m, c, float(eps),
                                              int(bool(zero_centered)), _code(x), _CODE[out_dtype], _stream()),
            "rmsnorm")
+    return out
+
+
+@_flushes
+def rmsnorm_pair(x, first, second, eps, zero_centered, out_dtype):
+    """Two RMSNorms of the same float32 rows [N, C] with weights of their own, in one pass over the rows."""
+    m, c = x.shape
+    for w in (first, second):
+        if w.dtype != torch.float32 or w.numel() != c or not w.is_contiguous():
+            raise ValueError("rmsnorm_pair takes dense float32 weights, one number per channel")
+    if x.dtype != torch.float32:
+        raise TypeError("rmsnorm_pair takes float32 rows")
+    outs = torch.empty((m, c), dtype=out_dtype, device=x.device), torch.empty((m, c), dtype=out_dtype, device=x.device)
+    _check(_fn("elementwise", "akas_rmsnorm_pair")(_ptr(_dense(x, "x")), _ptr(first), _ptr(second), _ptr(outs[0]), _ptr(outs[1]), m, c,
+                                                  float(eps), int(bool(zero_centered)), _CODE[out_dtype], _stream()), "rmsnorm_pair")
+    return outs
+
+
+@_flushes
+def round_rows(x, out):
+    """out[...] = x rounded to out's dtype, for dense float32 x [N, C] and ``out`` [N, C] whose rows may be parts of wider rows."""
+    n, c = x.shape
+    if x.dtype != torch.float32 or out.shape != x.shape:
+        raise ValueError("round_rows takes float32 x [N, C] and an output of its shape")
+    op, ldo = _rows(out, "out")
+    _check(_fn("elementwise", "akas_round_rows")(_ptr(_dense(x, "x")), op, ldo if n > 1 else max(ldo, c), n, c, _code(out), _stream()),
+           "round_rows")
     return out
 
 
@@ -984,6 +1016,32 @@ def norm_linear(h, norm_weight, eps, zero_centered, w, out_dtype=None, rows=None
     return linear_swiglu(x, w) if swiglu_out else linear(x, w, out_dtype=out_dtype)
 
 
+def absorbs_norm(h, w) -> bool:
+    """Whether ``norm_linear(h, ..., w)`` computes the norm on the product's way in (few tokens) instead of by itself."""
+    m, k = h.shape
+    return (w.dtype == torch.bfloat16 and h.dtype == torch.float32 and h.is_contiguous()
+            and (_chain_open or decode_products == "stream" or _skinny_fits(m, k)))
+
+
+def norm_linear_gated(h, norm_weight, eps, zero_centered, w_gate_up, width, bias, activation, rows=None):
+    """``linear_gated(rmsnorm(h[rows]), ...)`` for few tokens, the norm computed on the product's way in. None where the
+    fused kernel does not take the sizes or the dtype (the caller then runs the norm by itself)."""
+    m = rows.numel() if rows is not None else h.shape[0]
+    k, o = h.shape[1], w_gate_up.shape[0]
+    if activation not in _ACTIVATIONS:
+        raise ValueError(f"unknown activation {activation!r}")
+    if (w_gate_up.dtype != torch.bfloat16 or h.dtype != torch.float32 or not h.is_contiguous() or w_gate_up.shape[1] != k
+            or o != 2 * width or _chain_open or decode_products != "skinny" or products == "library" or not _skinny_fits(m, k)):
+        return None
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != o or not bias.is_contiguous()):
+        raise ValueError("norm_linear_gated takes a dense float32 bias [2F]")
+    out = torch.empty((m, width), dtype=torch.bfloat16, device=h.device)
+    _check(_fn("skinny_gemm", "akas_skinny_gemm_norm_gated")(_ptr(h), _ptr(rows), _ptr(norm_weight), float(eps), int(bool(zero_centered)),
+                                                            _ptr(_dense(w_gate_up, "w")), _ptr(out), m, o, k, _ptr(bias),
+                                                            _READOUT_ACTIVATIONS[activation], _stream()), "skinny gated product behind a norm")
+    return out
+
+
 # A decode step's in projection and gated short convolution as one kernel (csrc/skinny_gemm.cu, read-out "conv"):
 # AKAS_B200_FUSED_CONV=0 runs them as the product and the convolution kernel.
 fused_conv = os.environ.get("AKAS_B200_FUSED_CONV", "1") != "0"
@@ -1483,7 +1541,7 @@ def decay_scan(q, k, v, decay, state, cu_seqlens, slots, heads, dim, vdim, q_sca
 @_flushes
 def qk_norm_store(q, k, v, heads, kv_heads, dim, vdim, q_weight, k_weight, eps, k_pool, v_pool, block_table,
                   seq_of_token, positions, page_size, write=True, cos=None, sin=None, interleaved=False,
-                  q_bias=None, k_bias=None, v_bias=None):
+                  q_bias=None, k_bias=None, v_bias=None, unit_eps=None):
     n = q.shape[0]
     if not (q.dtype == k.dtype == v.dtype) or k_pool.dtype != v_pool.dtype:
         raise TypeError("qk_norm_store: q, k, v must have one dtype, and so must the pages")
@@ -1498,13 +1556,17 @@ def qk_norm_store(q, k, v, heads, kv_heads, dim, vdim, q_weight, k_weight, eps, 
         if cos.dtype != torch.float32 or sin.shape != cos.shape or cos.shape[0] != n or rot > dim:
             raise ValueError("qk_norm_store: rotary tables must be float32 [N, rot / 2] with rot <= dim")
         _dense(cos, "cos"), _dense(sin, "sin")
+    if unit_eps is not None:
+        if q_weight is not None or k_weight is not None:
+            raise ValueError("qk_norm_store norms in front of the rotation with weights or behind it without")
+        eps = unit_eps
     (qp, ldq), (kp, ldk), (vp, ldv) = _rows(q, "q"), _rows(k, "k"), _rows(v, "v")
     out = torch.empty((n, heads * dim), dtype=k_pool.dtype, device=q.device)
     _check(_fn("attention_general", "akas_qk_norm_store")(
         qp, ldq, kp, ldk, vp, ldv, _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(out), _ptr(k_pool), _ptr(v_pool),
         _ptr(block_table), block_table.shape[1], _ptr(seq_of_token), _ptr(positions), page_size, n, heads, kv_heads, dim, vdim,
         int(bool(write)), _code(k_pool), _ptr(cos), _ptr(sin), rot, int(bool(interleaved)), _code(q), _ptr(q_bias), _ptr(k_bias),
-        _ptr(v_bias), _stream()), "qk_norm_store")
+        _ptr(v_bias), int(unit_eps is not None), _stream()), "qk_norm_store")
     return out
 
 
@@ -1762,10 +1824,10 @@ def _shared_args(shared, n, c):
     return _ptr(y), _ptr(gate), gate.stride(0)
 
 
-def _moe_experts_grouped(h, w_gate_up, w_down, chosen, weights, update=None, weight_input=False, shared=None):
+def _moe_experts_grouped(h, w_gate_up, w_down, chosen, weights, update=None, weight_input=False, shared=None, activation=None):
     n, c = h.shape
     experts, f2, _ = w_gate_up.shape
-    f, top = f2 // 2, chosen.shape[1]
+    f, top = f2 // (2 if activation is None else 1), chosen.shape[1]
     hp, ldh = _rows(h, "h")
     cap = int(_fn("moe_grouped", "akas_moe_grouped_rows")(n * top, experts))
     dev = h.device
@@ -1780,9 +1842,10 @@ def _moe_experts_grouped(h, w_gate_up, w_down, chosen, weights, update=None, wei
                                               n, top, c, experts, _ptr(weights) if weight_input else None, _stream()),
            "moe_sort", kernels=2)
     gemm = _fn("moe_grouped", "akas_moe_grouped_gemm")
-    _check(gemm(_ptr(rows), _ptr(w_gate_up), _ptr(act), _ptr(tile_expert), _ptr(plan), cap, experts, f2, c, 2, _stream()),
+    _check(gemm(_ptr(rows), _ptr(w_gate_up), _ptr(act), _ptr(tile_expert), _ptr(plan), cap, experts, f2, c,
+                2 if activation is None else 4, _READOUT_PLAIN[activation] if activation is not None else 0, _stream()),
            "grouped gate and up product")
-    _check(gemm(_ptr(act), _ptr(w_down), _ptr(y), _ptr(tile_expert), _ptr(plan), cap, experts, c, f, 1, _stream()),
+    _check(gemm(_ptr(act), _ptr(w_down), _ptr(y), _ptr(tile_expert), _ptr(plan), cap, experts, c, f, 1, 0, _stream()),
            "grouped down product")
     _check(_fn("moe_grouped", "akas_moe_combine")(hp, ldh, _ptr(y), _ptr(row_of_pair), None if weight_input else _ptr(weights),
                                                  _ptr(out), n, top, c, *_update_args(update, n, c), *_shared_args(shared, n, c),
@@ -1791,26 +1854,30 @@ def _moe_experts_grouped(h, w_gate_up, w_down, chosen, weights, update=None, wei
 
 
 @_flushes
-def moe_experts(h, w_gate_up, w_down, chosen, weights, update=None, weight_input=False, shared=None):
+def moe_experts(h, w_gate_up, w_down, chosen, weights, update=None, weight_input=False, shared=None, activation=None):
     """``weight_input``: the weight multiplies the expert's input, sum_k expert(w_k h), where otherwise it multiplies the
     result. ``shared`` = (y float32 [N, C], gate float32 [N, 1] or None): y times its gate is added to the sum.
     The weighted sum of the chosen experts' results, float32 [N, C]. With ``update`` = (x, a, scale_a, scale_b, mult)
     the sum is not returned but added into the residual stream by the last kernel: x += mult * (scale_a * a + scale_b *
-    sum), in place; returns x."""
+    sum), in place; returns x. ``activation`` ("relu2", "gelu_tanh", "silu"; None: gated experts): experts without a gate,
+    w_gate_up = w_up [E, F, C]."""
     n, c = h.shape
     experts, f2, _ = w_gate_up.shape
-    f, top = f2 // 2, chosen.shape[1]
+    f, top = f2 // (2 if activation is None else 1), chosen.shape[1]
+    if activation is not None and activation not in _READOUT_PLAIN:
+        raise ValueError(f"unknown activation {activation!r}")
     if w_gate_up.dtype != h.dtype or w_down.dtype != h.dtype or w_down.shape != (experts, c, f) or w_gate_up.shape[2] != c:
-        raise ValueError("moe_experts takes h [N, C], w_gate_up [E, 2 F, C] and w_down [E, C, F] of one dtype")
+        raise ValueError("moe_experts takes h [N, C], w_gate_up [E, 2 F, C] (or w_up [E, F, C]) and w_down [E, C, F] of one dtype")
     hp, ldh = _rows(h, "h")
     if (moe_kernels == "auto" and h.dtype == torch.bfloat16 and n * top > _MOE_SIMPLE_PAIRS and ldh % 8 == 0 and hp % 16 == 0
             and _fn("moe_grouped", "akas_moe_grouped_takes")(c, f, experts)):
         _dense(w_gate_up, "w_gate_up"), _dense(w_down, "w_down")
-        return _moe_experts_grouped(h, w_gate_up, w_down, chosen, weights, update, weight_input, shared)
+        return _moe_experts_grouped(h, w_gate_up, w_down, chosen, weights, update, weight_input, shared, activation)
     act = torch.empty((n * top, f), dtype=h.dtype, device=h.device)
     out = torch.empty((n, c), dtype=torch.float32, device=h.device) if update is None else update[0]
     _check(_fn("moe", "akas_moe_gate_up")(hp, ldh, _ptr(_dense(w_gate_up, "w_gate_up")), _ptr(chosen), _ptr(act), n, top, c, f,
-                                         experts, _code(h), _ptr(weights) if weight_input else None, _stream()), "moe_gate_up")
+                                         experts, _code(h), _ptr(weights) if weight_input else None,
+                                         _READOUT_PLAIN[activation] if activation is not None else 0, _stream()), "moe_gate_up")
     _check(_fn("moe", "akas_moe_down")(hp, ldh, _ptr(_dense(w_down, "w_down")), _ptr(chosen), None if weight_input else _ptr(weights),
                                       _ptr(act), _ptr(out), n, top, c, f, experts, _code(h), *_update_args(update, n, c),
                                       *_shared_args(shared, n, c), _stream()), "moe_down")

@@ -37,6 +37,17 @@ def rmsnorm(x, weight, eps, zero_centered, out_dtype, rows=None):
     return y.to(out_dtype)
 
 
+def rmsnorm_pair(x, first, second, eps, zero_centered, out_dtype):
+    """Two RMSNorms of the same rows with weights of their own, one eps and one meaning of the weight."""
+    return rmsnorm(x, first, eps, zero_centered, out_dtype), rmsnorm(x, second, eps, zero_centered, out_dtype)
+
+
+def round_rows(x, out):
+    """out[...] = x rounded to out's dtype, for float32 x [N, C] and ``out`` [N, C] whose rows may be parts of wider rows."""
+    out.copy_(x)
+    return out
+
+
 def linear(x, w, out_dtype=None, residual=None, bias=None):
     """x [N, K] times w [O, K] transposed, float32 accumulation, plus ``bias`` (float32 [O]) where one is given, before
     the one rounding; ``residual`` (float32) is added to in place."""
@@ -405,12 +416,13 @@ def gated_rmsnorm(o, weight, eps, gate, heads, vdim, out_dtype, gate_activation=
 
 def qk_norm_store(q, k, v, heads, kv_heads, dim, vdim, q_weight, k_weight, eps, k_pool, v_pool, block_table,
                   seq_of_token, positions, page_size, write=True, cos=None, sin=None, interleaved=False,
-                  q_bias=None, k_bias=None, v_bias=None):
+                  q_bias=None, k_bias=None, v_bias=None, unit_eps=None):
     """First, where biases (float32 [heads * dim], [kv_heads * dim], [kv_heads * vdim]) are given, q, k and v plus
     their biases (q, k and v may then be float32 results of a product, rounded here for the first time). Then
     per-head RMSNorm (plain weight; None: no norm) of q [N, heads * dim] and k [N, kv_heads * dim], then, where
     ``cos`` and ``sin`` (float32 [N, rot / 2]) are given, the rotation of the first ``rot`` channels of every head of
-    q and k: channel 2i with 2i + 1 (``interleaved``) or i with i + rot / 2. k and the untouched v [N, kv_heads * vdim]
+    q and k: channel 2i with 2i + 1 (``interleaved``) or i with i + rot / 2. Then, where ``unit_eps`` is given, every
+    head of q and k over sqrt(mean of its dim squares + unit_eps), without a weight. k and the untouched v [N, kv_heads * vdim]
     go into the pages (k pages [.., kv_heads, page, dim], v pages [.., kv_heads, page, vdim]); returns q, contiguous,
     in the pools' dtype."""
     n = q.shape[0]
@@ -446,6 +458,8 @@ def qk_norm_store(q, k, v, heads, kv_heads, dim, vdim, q_weight, k_weight, eps, 
             return x
 
         qf, kf = turn(qf), turn(kf)
+    if unit_eps is not None:
+        qf, kf = (x * torch.rsqrt((x * x).mean(dim=-1, keepdim=True) + unit_eps) for x in (qf, kf))
     if write:
         live, page, off = _page_addresses(block_table, seq_of_token, positions, page_size)
         k_pool[page[live], :, off[live]] = kf[live].to(k_pool.dtype)
@@ -629,8 +643,8 @@ def moe_route(h, w_router, correction, groups, keep, top, scoring="softmax", ren
     score is their largest choice score, and only outputs of the ``keep`` best groups can be chosen; the ``top``
     largest choice scores win (ties: the lower index). Returns (chosen int32 [N, top], weights float32 [N, top]): the
     chosen outputs in the order of their choice scores and their plain scores over their sum (+ 1e-20).
-    ``scoring="sigmoid"``: a score is the sigmoid of its logit (without a correction the choice goes by the logits, which
-    order the same way); ``correction`` None: none; ``renormalize`` False: the
+    Without a correction the choice goes by the logits, which order as the scores do. ``scoring="sigmoid"``: a score is
+    the sigmoid of its logit; ``correction`` None: none; ``renormalize`` False: the
     weights are the chosen scores as they are. ``extra`` = X > 0: w_router has X more rows [R + X, C] that take no part
     in the choice; the sigmoids of their logits are returned as a third result, float32 [N, X]."""
     n = h.shape[0]
@@ -639,8 +653,8 @@ def moe_route(h, w_router, correction, groups, keep, top, scoring="softmax", ren
     s = torch.softmax(z[:, :r], dim=-1) if scoring == "softmax" else torch.sigmoid(z[:, :r])
     if correction is not None:
         pick = s + correction.to(torch.float32)
-    else:  # the logits order as their scores do, and still compare where two sigmoids round to one
-        pick = z[:, :r].clone() if scoring == "sigmoid" else s
+    else:  # the logits order as their scores do, and still compare where two scores round to one
+        pick = z[:, :r].clone()
     if groups > 1 and keep < groups:
         best = pick.reshape(n, groups, r // groups).max(dim=-1).values
         order = torch.argsort(best, dim=-1, descending=True, stable=True)
@@ -656,8 +670,9 @@ def moe_route(h, w_router, correction, groups, keep, top, scoring="softmax", ren
     return chosen.to(torch.int32), w
 
 
-def moe_experts(h, w_gate_up, w_down, chosen, weights, update=None, weight_input=False, shared=None):
-    """``weight_input``: the weight multiplies the expert's input, out[n] = sum_k expert(weights[n, k] h[n]) (computed
+def moe_experts(h, w_gate_up, w_down, chosen, weights, update=None, weight_input=False, shared=None, activation=None):
+    """``activation`` (None: gated experts as below): experts without a gate, w_down[e] act(w_up[e] h) with w_gate_up =
+    w_up [E, F, C] and act "relu2", "gelu_tanh" or "silu". ``weight_input``: the weight multiplies the expert's input, out[n] = sum_k expert(weights[n, k] h[n]) (computed
     as silu(w g) * (w u) on the float32 sums g, u of the unweighted row). ``shared`` = (y float32 [N, C], gate float32
     [N, 1] or None): y, times its gate, is added to the sum. With ``update`` = (x, a, scale_a, scale_b, mult): x += mult * (scale_a * a + scale_b * out) in place, returns x. Else
     out[n] = sum_k weights[n, k] * expert_(chosen[n, k])(h[n]) in float32 [N, C]. Expert e < E computes
@@ -677,7 +692,11 @@ def moe_experts(h, w_gate_up, w_down, chosen, weights, update=None, weight_input
             gu = hf[rows] @ w_gate_up[e].to(torch.float32).T
             if weight_input:
                 gu, g = gu * g, 1.0
-            act = (torch.nn.functional.silu(gu[:, : f2 // 2]) * gu[:, f2 // 2 :]).to(h.dtype).to(torch.float32)
+            if activation is not None:
+                act = _activation(gu, activation)
+            else:
+                act = torch.nn.functional.silu(gu[:, : f2 // 2]) * gu[:, f2 // 2 :]
+            act = act.to(h.dtype).to(torch.float32)
             out[rows] += g * (act @ w_down[e].to(torch.float32).T)
     if shared is not None:
         y, gate = shared

@@ -11,7 +11,8 @@ and to itself; the output product, added to the residual.
 A layer whose spec asks for more than that (value heads of another size than the keys', a capped score, a
 logarithmic distance penalty, first tokens kept behind the window, a sink in the softmax's denominator (exp(0) or a
 learned logit per head), a gate per head on the output, values that are the keys as projected, rotary pairs of
-neighbouring channels, biases on q, k and v, no keys and values of its own but another layer's cache) runs the same
+neighbouring channels, biases on q, k and v, heads of q and k divided by their root mean square after the position
+encoding, no keys and values of its own but another layer's cache) runs the same
 steps on the general kernels: one product for q, k, v and the gate's
 logits, QK-norm, rotation and page write (``ops.qk_norm_store``), attention with the options as arguments
 (``ops.attention_general``), the output product. ``core`` is that sequence without the two products, for a mixer
@@ -53,6 +54,9 @@ class Attention(Mixer):
             raise ValueError(f"unknown output gate {s.gate!r}; known: 'head', 'channel'")
         if self.general and s.keep_first and not s.window:
             raise ValueError("keep_first needs a window")
+        self.unit_eps = getattr(s, "qk_unit_eps", None)
+        if self.unit_eps is not None and s.qk_norm is not None:
+            raise ValueError("q and k are normed in front of the position encoding (qk_norm) or behind it (qk_unit_eps), not both")
         self.own_kv = bool(getattr(s, "own_kv", True))
         self.biased = bool(getattr(s, "bias", False))
         if not self.own_kv and getattr(s, "values_are_keys", False):
@@ -166,10 +170,10 @@ class Attention(Mixer):
         if norm is not None and norm.zero_centered:
             raise ValueError("the general attention kernels take a plain QK-norm weight")
         table = ctx.block_table(cache.group)
-        rotary = {}
+        rotary = {} if self.unit_eps is None else dict(unit_eps=self.unit_eps)
         if self.position is not None:
             cos, sin = self.position.tables(ctx)
-            rotary = dict(cos=cos, sin=sin, interleaved=self.position.interleaved)
+            rotary.update(cos=cos, sin=sin, interleaved=self.position.interleaved)
         if self.bias is not None:
             rotary.update(q_bias=self.bias[:nq], k_bias=self.bias[nq : nq + nk] if nk else None,
                           v_bias=self.bias[nq + nk : nq + nk + nv] if nv else None)

@@ -143,11 +143,30 @@ class Normed:
     def __init__(self, norm, h, rows=None):
         self.norm, self.h, self.rows = norm, h, rows
         self._tensor = None
+        self.partner: Optional["Normed"] = None  # another norm of the same rows, made with this one in one pass (norm_pair)
+        self.absorbed = False  # a product has computed the norm on its way in: nobody wants the tensor
 
     def tensor(self):
         if self._tensor is None:
-            self._tensor = self.norm.forward(self.h, rows=self.rows)
+            other = self.partner
+            if other is not None and other._tensor is None and not other.absorbed:
+                spec = self.norm.spec
+                self._tensor, other._tensor = self.norm.rt.ops.rmsnorm_pair(
+                    self.h, self.norm.weight, other.norm.weight, spec.eps, spec.zero_centered, self.norm.rt.dtype)
+            else:
+                self._tensor = self.norm.forward(self.h, rows=self.rows)
         return self._tensor
+
+
+def norm_pair(first, second, h):
+    """Two norms of the same rows that have not run yet. Two RMSNorms with the same eps read the rows once where the
+    operations offer that, unless a product takes one of them in."""
+    a, b = Normed(first, h), Normed(second, h)
+    sa, sb = first.spec, second.spec
+    alike = all(getattr(sa, f, None) == getattr(sb, f, None) for f in ("kind", "eps", "zero_centered"))
+    if alike and getattr(sa, "kind", None) == "rmsnorm" and hasattr(first.rt.ops, "rmsnorm_pair"):
+        a.partner, b.partner = b, a
+    return a, b
 
 
 def project(rt: "Runtime", x, w, out_dtype=None, residual=None, bias=None):
@@ -156,7 +175,8 @@ def project(rt: "Runtime", x, w, out_dtype=None, residual=None, bias=None):
     if isinstance(x, Normed):
         spec = x.norm.spec
         kind = getattr(spec, "kind", None)
-        if residual is None and bias is None and kind == "rmsnorm" and hasattr(rt.ops, "norm_linear"):
+        if residual is None and bias is None and kind == "rmsnorm" and _takes_norm(rt.ops, x, w):
+            x.absorbed = True
             return rt.ops.norm_linear(x.h, x.norm.weight, spec.eps, spec.zero_centered, w, out_dtype, x.rows)
         if residual is None and bias is None and kind == "dynamic_tanh" and hasattr(rt.ops, "dyt_linear"):
             out = rt.ops.dyt_linear(x.h, x.norm.alpha, x.norm.weight, x.norm.shift, w, out_dtype, x.rows)
@@ -168,6 +188,14 @@ def project(rt: "Runtime", x, w, out_dtype=None, residual=None, bias=None):
     return rt.ops.linear(x, w, out_dtype=out_dtype, residual=residual)
 
 
+def _takes_norm(ops, x: Normed, w) -> bool:
+    """Whether ``ops.norm_linear`` should have this norm: always for a norm that stands alone; one of a pair only where
+    the product really computes it on its way in (else the pair's one pass is the cheaper way)."""
+    if not hasattr(ops, "norm_linear"):
+        return False
+    return x._tensor is None and (x.partner is None or (hasattr(ops, "absorbs_norm") and ops.absorbs_norm(x.h, w)))
+
+
 def project_gated(rt: "Runtime", x, w_gate_up, width, bias, activation):
     """``act(x . w_g^T + b_g) * (x . w_u^T + b_u)`` for the stacked ``[w_g; w_u]`` (``width`` rows each), for a tensor or a ``Normed``: in the
     read-out of the product where the kernels offer that, else the product in float32 and the activation's kernel."""
@@ -176,6 +204,12 @@ def project_gated(rt: "Runtime", x, w_gate_up, width, bias, activation):
         if getattr(x.norm.spec, "kind", None) == "dynamic_tanh" and hasattr(ops, "dyt_linear"):
             out = ops.dyt_linear(x.h, x.norm.alpha, x.norm.weight, x.norm.shift, w_gate_up, None, x.rows, gated=(width, bias, activation))
             if out is not None:
+                return out
+        if getattr(x.norm.spec, "kind", None) == "rmsnorm" and hasattr(ops, "norm_linear_gated"):
+            spec = x.norm.spec
+            out = ops.norm_linear_gated(x.h, x.norm.weight, spec.eps, spec.zero_centered, w_gate_up, width, bias, activation, x.rows)
+            if out is not None:
+                x.absorbed = True
                 return out
         x = x.tensor()
     if hasattr(ops, "linear_gated"):

@@ -2,8 +2,10 @@
 
 ``pre_norm`` (the only arrangement LFM2 uses, src/akas/models/lfm2/_composition.py:189,308-309,356
 in kreasof-ai/akas): h += mixer(norm(h)); h += ffn(norm(h)). ``parallel``: one norm n = norm(h) that the mixer and
-the feed-forward both read, h += m * (s1 * mixer(n) + s2 * ffn(n)) with a constant m and a learned scale per channel
-for each sublayer (the two results are float32 and meet the residual stream in one kernel). ``sandwich``: a norm in
+the feed-forward both read, or a norm for each, both of the same h; h += m * (s1 * mixer(n) + s2 * ffn(n)) with a
+constant m and a learned scale per channel for each sublayer (the two results are float32 and meet the residual stream
+in one kernel; without constant and scales, a feed-forward in two halves adds into the stream like the mixer does, both
+once everything that reads the stream has run). ``sandwich``: a norm in
 front of and a norm behind each sublayer, h += post(mixer(norm(h))); h += post(ffn(norm(h))), the sublayers' results
 float32, the second norm and the sum one kernel where the norm offers that (``add_to``). Other arrangements are
 added to ``ARRANGEMENTS`` as functions of (block, h, ctx, cache, write).
@@ -13,7 +15,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import Param, Runtime, build_part, load_norm, norm_params
+from .base import Param, Runtime, build_part, load_norm, norm_pair, norm_params
 
 
 def _normed(norm, part, h):
@@ -37,7 +39,34 @@ def _float32_result(part, *args, **kwargs):
     return part.forward(*args, **kwargs).to(torch.float32)
 
 
+def _given(part, normed):
+    """A norm that has not run yet as ``part`` takes it."""
+    return normed if getattr(part, "takes_normed", False) else normed.tensor()
+
+
+def _parallel_two_norms(block, h, ctx, cache, write):
+    mixer, ffn = block.mixer, block.ffn
+    n1, n2 = norm_pair(block.mixer_norm, block.ffn_norm, h)
+    plain = block.mixer_scale is None and block.ffn_scale is None and block.spec.residual_multiplier == 1.0
+    if plain and hasattr(ffn, "begin"):
+        # Everything that reads h runs before anything adds into it: the feed-forward's first half behind its norm, then
+        # the mixer, whose norm rides in (or ran beside the other) and whose output product adds into h; then the
+        # feed-forward's output product does. No sublayer's result is written by itself.
+        held = ffn.begin(_given(ffn, n2), ctx)
+        h = mixer.forward(_given(mixer, n1), ctx, cache, residual=h, write=write)
+        return ffn.finish(held, residual=h)
+    a = _float32_result(mixer, _given(mixer, n1), ctx, cache, residual=None, write=write)
+    if hasattr(ffn, "forward_update"):
+        return ffn.forward_update(n2.tensor(), ctx, h, a, block.mixer_scale, block.ffn_scale, block.spec.residual_multiplier)
+    b = _float32_result(ffn, _given(ffn, n2), ctx, residual=None)
+    return mixer.rt.ops.scaled_add(h, a, block.mixer_scale, b, block.ffn_scale, block.spec.residual_multiplier)
+
+
 def _parallel(block, h, ctx, cache, write):
+    if block.ffn is not None and block.ffn_norm is not None:
+        return _parallel_two_norms(block, h, ctx, cache, write)
+    if block.ffn is None and block.mixer_scale is None and block.spec.residual_multiplier == 1.0:
+        return block.mixer.forward(_normed(block.mixer_norm, block.mixer, h), ctx, cache, residual=h, write=write)
     n = block.mixer_norm.forward(h)
     a = _float32_result(block.mixer, n, ctx, cache, residual=None, write=write)
     if hasattr(block.ffn, "forward_update"):  # the feed-forward's last kernel does the block's update itself

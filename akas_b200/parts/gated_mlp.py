@@ -46,12 +46,20 @@ class GatedMLP(FeedForward):
             self.bias_gate_up = torch.cat([get(self._n("gate") + ".b"), get(self._n("up") + ".b")]).contiguous()
             self.bias_down = get(self._n("down") + ".b")
 
+    def begin(self, x, ctx):
+        """The half that reads the normed input: the hidden activations, for ``finish``."""
+        return project_gated(self.rt, x, self.w_gate_up, self.spec.intermediate_size, self.bias_gate_up, self.spec.activation)
+
+    def finish(self, act, residual):
+        """The half that adds the down product into the residual stream."""
+        return project(self.rt, act, self.w_down, residual=residual, bias=self.bias_down)
+
     def forward(self, x, ctx, residual=None):
-        act = project_gated(self.rt, x, self.w_gate_up, self.spec.intermediate_size, self.bias_gate_up, self.spec.activation)
+        act = self.begin(x, ctx)
         if residual is None:
             out = project(self.rt, act, self.w_down, out_dtype=torch.float32, bias=self.bias_down)
             return out.to(self.rt.dtype)
-        return project(self.rt, act, self.w_down, residual=residual, bias=self.bias_down)
+        return self.finish(act, residual)
 
 
 register_ffn("gated_mlp", GatedMLP)

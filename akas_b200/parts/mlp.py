@@ -51,8 +51,16 @@ class MLP(FeedForward):
     def load(self, get):
         self.w_up, self.w_down = get(self._n("up")), get(self._n("down"))
 
+    def begin(self, x, ctx):
+        """The half that reads the normed input: the hidden activations, for ``finish``."""
+        return project_activated(self.rt, x, self.w_up, self.spec.activation)
+
+    def finish(self, act, residual):
+        """The half that adds the down product into the residual stream."""
+        return project(self.rt, act, self.w_down, residual=residual)
+
     def forward(self, x, ctx, residual=None, out_dtype=None):
-        act = project_activated(self.rt, x, self.w_up, self.spec.activation)
+        act = self.begin(x, ctx)
         return project(self.rt, act, self.w_down, out_dtype=out_dtype, residual=residual)
 
 

@@ -1,4 +1,4 @@
-"""A routed feed-forward: a mixture of SwiGLU experts, a few per token, some of them identities.
+"""A routed feed-forward: a mixture of experts (SwiGLU, or ungated with a plain activation), a few per token, some of them identities.
 
 Per token (all of the router in float32): scores = softmax(W_router x) over every router output; the choice goes by
 score + correction among the outputs of the best groups of neighbours; the weights are the chosen outputs' plain
@@ -10,7 +10,8 @@ number.
 Options of the spec change the rule: sigmoid scores instead of a softmax, no correction, weights that are the chosen
 scores as they are, a weight that multiplies the expert's input (sum expert(w x)) instead of its result, and one more
 expert that every token passes, whose result is added to the sum, times sigmoid(W_sg x) (one number per token) where
-the spec says so. That expert is a gated feed-forward on the products' own kernels; its gate's logit is one more row
+the spec says so; experts without a gate matrix, W_down act(W_up x), whose stack is then [experts, F, C]. The expert
+that every token passes is a feed-forward on the products' own kernels, with the activation in their read-out; its gate's logit is one more row
 of the router's float32 matrix, and the experts' last kernel adds its result to theirs.
 """
 
@@ -19,6 +20,7 @@ from __future__ import annotations
 import torch
 
 from .base import FeedForward, Param, project, project_gated, register_ffn, renamed, stack_rows
+from .mlp import ACTIVATIONS, project_activated
 
 
 class RoutedExperts(FeedForward):
@@ -47,6 +49,10 @@ class RoutedExperts(FeedForward):
             raise ValueError("a weight on the expert's input leaves identity experts without a rule")
         self.shared_size = getattr(s, "shared_size", None)
         self.shared_gate = bool(getattr(s, "shared_gate", False)) and self.shared_size is not None
+        self.gated = bool(getattr(s, "gated", True))
+        self.activation = getattr(s, "activation", "silu")
+        if self.activation not in (("silu",) if self.gated else ACTIVATIONS):
+            raise ValueError(f"unknown activation {self.activation!r} of {'gated' if self.gated else 'ungated'} experts")
         self.has_correction = bool(getattr(s, "correction", True))
         self.renormalize = bool(getattr(s, "renormalize", True))
         # the plain rule keeps the call it always made; anything else names its options
@@ -66,13 +72,15 @@ class RoutedExperts(FeedForward):
             p[self._n("correction")] = Param((outputs,), role="vector")
         if self.shared_size is not None:
             fs = self.shared_size
-            p[self._n("shared.gate")] = Param((fs, c))
+            if self.gated:
+                p[self._n("shared.gate")] = Param((fs, c))
             p[self._n("shared.up")] = Param((fs, c))
             p[self._n("shared.down")] = Param((c, fs))
             if self.shared_gate:
                 p[self._n("shared.sg")] = Param((1, c), role="vector")
         for e in range(s.num_experts):
-            p[self._n(f"e{e}.gate")] = Param((f, c))
+            if self.gated:
+                p[self._n(f"e{e}.gate")] = Param((f, c))
             p[self._n(f"e{e}.up")] = Param((f, c))
             p[self._n(f"e{e}.down")] = Param((c, f))
         return p
@@ -82,11 +90,13 @@ class RoutedExperts(FeedForward):
         self.w_router = get(self._n("router"))
         self.correction = get(self._n("correction")) if self.has_correction else None
         if self.shared_size is not None:
-            self.w_shared_gate_up = stack_rows([get(self._n("shared.gate")), get(self._n("shared.up"))])
+            halves = ("gate", "up") if self.gated else ("up",)
+            self.w_shared_gate_up = stack_rows([get(self._n(f"shared.{half}")) for half in halves], 16 if self.gated else 1)
             self.w_shared_down = get(self._n("shared.down"))
             if self.shared_gate:  # the gate's logit is one more output of the router's product
                 self.w_router = torch.cat([self.w_router, get(self._n("shared.sg")).reshape(1, -1)], dim=0).contiguous()
         self.w_gate_up = torch.stack(
+            [get(self._n(f"e{e}.up")) for e in range(s.num_experts)] if not self.gated else
             [torch.cat([get(self._n(f"e{e}.gate")), get(self._n(f"e{e}.up"))], dim=0) for e in range(s.num_experts)]
         ).contiguous()
         self.w_down = torch.stack([get(self._n(f"e{e}.down")) for e in range(s.num_experts)]).contiguous()
@@ -106,10 +116,15 @@ class RoutedExperts(FeedForward):
         more = {}
         if self.weight_input:
             more["weight_input"] = True
+        if not self.gated:
+            more["activation"] = self.activation
         if self.shared_size is not None:
-            # the expert that every token passes: a gated feed-forward on the products' kernels, float32 out; the
-            # experts' last kernel adds it, times its gate
-            act = project_gated(self.rt, x, self.w_shared_gate_up, self.shared_size, None, "silu")
+            # the expert that every token passes: a feed-forward on the products' kernels, float32 out; the experts'
+            # last kernel adds it, times its gate
+            if self.gated:
+                act = project_gated(self.rt, x, self.w_shared_gate_up, self.shared_size, None, "silu")
+            else:
+                act = project_activated(self.rt, x, self.w_shared_gate_up, self.activation)
             more["shared"] = (project(self.rt, act, self.w_shared_down, out_dtype=torch.float32), gate)
         return ops.moe_experts(x, self.w_gate_up, self.w_down, chosen, weights, update=update, **more)
 
