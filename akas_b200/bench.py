@@ -59,6 +59,9 @@ def prefill_flops(runner: ModelRunner, tokens: int, start: int = 0) -> float:
     p = matrix_params(runner)
     flops = 2.0 * tokens * p["layers"] + 2.0 * p["head"]
     for entry in runner.model.schedule:
+        if entry.join is not None:  # the matrix that joins the embedding's output to the stream
+            flops += 2.0 * tokens * runner.model.joins[entry.join].numel()
+    for entry in runner.model.schedule:
       for spec in _mixer_specs(runner.model.blocks[entry.layer].mixer.spec):
         kind = getattr(spec, "kind", "")
         if kind == "attention":
@@ -523,6 +526,25 @@ def kidarax_shape_config(name: str) -> dict:
                 loop=dict(start=runs // 2 - 2, stop=runs // 2, times=2), layers=layers)
 
 
+# Pekodra at LFM2's layer sizes: the same width and vocabulary; fourteen layers of which two run twice (a loop), so sixteen
+# layer runs like LFM2's. Attention with LFM2's head counts inside a window of 1,024 in every layer; feed-forwards take
+# turns: a gated one with biases, two thirds as wide as LFM2's (the two matrices of Kidarax's hold as many parameters),
+# and sixteen ungated experts of three eighths of LFM2's width (as many parameters as three matrices of a quarter) of
+# which a token passes three, beside one more that every token passes.
+def pekodra_shape_config(name: str) -> dict:
+    lfm2 = config_from_shape(name)
+    c, ff3 = lfm2.hidden_size, lfm2.feed_forward_size
+    attention = dict(heads=lfm2.num_attention_heads, kv_heads=lfm2.num_key_value_heads, dim=lfm2.head_dim, vdim=lfm2.head_dim,
+                     scale=lfm2.head_dim ** -0.5, mask=dict(size=1024),
+                     rot=dict(base=500000.0, dims=lfm2.head_dim, scaling=dict(factor=8.0, original=4096, fast=32.0, slow=1.0)))
+    dense = dict(kind="dense", ff=2 * ff3 // 3 // 64 * 64)
+    moe = dict(kind="moe", expert=dict(ff=3 * ff3 // 8), router=dict(experts=16, top=3), shared=dict(ff=3 * ff3 // 8))
+    runs = len(lfm2.layer_kinds)
+    return dict(architecture="Pekodra", width=c, vocab=lfm2.vocab_size, norm=dict(eps=1e-5), embedding=dict(scale=float(c) ** 0.5),
+                logit_scale=float(c) ** -0.5, loop=dict(start=runs // 2 - 2, stop=runs // 2, times=2),
+                layers=[dict(type="attention", mixer=attention, mlp=moe if i % 2 else dense) for i in range(runs - 2)])
+
+
 def config_from_shape(name: str):
     from .config import config_from_dict
 
@@ -549,7 +571,7 @@ def compare_designs(shape: str = "1.2b", prompt: int = 2048, batches=(8, 64), st
 
     rows = []
     shapes = {"lfm2": shape_config, "gigusun": gigusun_shape_config, "girelix": girelix_shape_config,
-              "penopel": penopel_shape_config, "kidarax": kidarax_shape_config}
+              "penopel": penopel_shape_config, "kidarax": kidarax_shape_config, "pekodra": pekodra_shape_config}
     for design, data in ((name, shapes[name](shape)) for name in designs):
         say(f"{design} {shape}: writing random weights")
         model_config = config_from_dict(data)

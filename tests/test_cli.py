@@ -131,3 +131,29 @@ def test_generate_runs_a_kidarax_folder(tmp_path, capsys):
     for extra in ([], ["--temperature", "0.7", "--top-k", "20", "--seed", "2", "--dtype", "float32"]):
         main(["generate", "--model", str(tmp_path / "k"), "--prompt", "5 17 3 9", "--max-tokens", "7", "--ignore-eos", *extra])
         assert len(capsys.readouterr().out.split()) == 7
+
+
+def test_random_and_inspect_take_a_pekodra_configuration(tmp_path, capsys):
+    import tiny_pekodra
+
+    config = tiny_pekodra.CONFIGS["mix"]
+    main(["random", "--out", str(tmp_path / "k"), "--config", json.dumps(config), "--seed", "4"])
+    capsys.readouterr()
+    main(["inspect", "--model", str(tmp_path / "k")])
+    report = json.loads(capsys.readouterr().out)
+    assert report["architecture"] == "Pekodra" and report["config"] == json.loads(json.dumps(config))
+    assert {"loop.in", "head", "l0.norm1", "l0.norm2", "l0.mlp.router", "l0.mlp.e5.down", "l0.mlp.shared.up", "l1.mlp.gate.b",
+            "l1.mlp.down.b", "l3.mix.v", "final.norm"} <= set(report["inventory"])
+    # no gate matrices of experts, no shared gate, no biases in the mixer, no norm for a feed-forward that is not there
+    assert not {"l0.mlp.e0.gate", "l0.mlp.shared.sg", "l0.mix.q.b", "l3.mlp.up"} & set(report["inventory"])
+
+
+@pytest.mark.gpu
+def test_generate_runs_a_pekodra_folder(tmp_path, capsys):
+    import tiny_pekodra
+
+    main(["random", "--out", str(tmp_path / "k"), "--config", json.dumps(tiny_pekodra.CONFIGS["mix"]), "--seed", "4"])
+    capsys.readouterr()
+    for extra in ([], ["--temperature", "0.7", "--top-k", "20", "--seed", "2", "--dtype", "float32"]):
+        main(["generate", "--model", str(tmp_path / "k"), "--prompt", "5 17 3 9", "--max-tokens", "7", "--ignore-eos", *extra])
+        assert len(capsys.readouterr().out.split()) == 7
