@@ -119,7 +119,8 @@ class AttentionSpec:
         """Whether the layer needs what only the general attention kernels compute."""
         return bool(self.v_head_dim not in (None, self.head_dim) or self.softcap or self.distance_bias or self.keep_first
                     or self.sink or self.gate or self.values_are_keys or getattr(self.position, "interleaved", False)
-                    or self.bias or not self.own_kv or self.qk_unit_eps is not None)
+                    or self.bias or not self.own_kv
+                    or (self.qk_unit_eps is not None and self.head_dim not in (16, 32, 64, 128)))  # sizes of the tensor-core kernels
 
 
 @dataclass(frozen=True)

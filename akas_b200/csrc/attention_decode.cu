@@ -359,7 +359,7 @@ struct Fresh {
   const float* q_w;    // the norms' weights over a head (nullptr: no norm)
   const float* k_w;
   float eps;
-  int zero_centered;
+  int zero_centered;   // or AKAS_UNIT_BEHIND: no weights, the division by the root mean square behind the rotation
   const float* cos_t;  // [N, rotary / 2] each (nullptr: no rotation)
   const float* sin_t;
   int rotary;

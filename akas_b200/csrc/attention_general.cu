@@ -98,6 +98,102 @@ __global__ void qk_norm_store_kernel(const TI* __restrict__ q, long long ldq, co
   }
 }
 
+// The same for head sizes that are multiples of 8 (at most 256), rotate-half pairs and a rotary width that is a multiple
+// of 16, everything on 16 bytes: a thread owns 8 neighbouring channels of a head (LPH threads, D / 8 rounded up to a
+// power of two, share one; those past D / 8 only shuffle, as do those past the last head) and reads its rotation partner's 8 channels itself; the
+// threads behind the heads' copy the values. A token's heads are spread over gridDim.y blocks.
+template <typename TI, typename T>
+__global__ void __launch_bounds__(128)
+qk_norm_store8_kernel(const TI* __restrict__ q, long long ldq, const TI* __restrict__ k, long long ldk, const TI* __restrict__ v,
+                      long long ldv, const float* __restrict__ qw, const float* __restrict__ kw, float eps, T* __restrict__ q_out,
+                      T* __restrict__ k_pool, T* __restrict__ v_pool, const int* __restrict__ block_table, int max_blocks,
+                      const int* __restrict__ seq_of_token, const int* __restrict__ positions, int page_size, int H, int G, int D,
+                      int V, int write, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot,
+                      const float* __restrict__ qb, const float* __restrict__ kb, const float* __restrict__ vb, int unit, int lph) {
+  const int n = blockIdx.x;
+  const int req = seq_of_token[n];
+  if (req < 0) return;
+  const int item = blockIdx.y * blockDim.x + threadIdx.x;
+  const int heads = write ? H + G : H;
+  const int head = item / lph, e0 = item % lph * 8;
+  const bool turns = head < heads && e0 < D;
+  const bool is_q = head < H;
+  long long row = 0;  // the token's row in a pool of one head
+  if (write && head >= H) {
+    const int pos = positions[n];
+    row = (long long)block_table[(size_t)req * max_blocks + pos / page_size] * G * page_size + pos % page_size;
+  }
+  float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  const int g = head - H;
+  const float* w = is_q ? qw : kw;
+  const TI* src = is_q ? q + (size_t)n * ldq + (size_t)head * D : k + (size_t)n * ldk + (size_t)g * D;
+  const float* bias = is_q ? (qb != nullptr ? qb + (size_t)head * D : nullptr) : (kb != nullptr ? kb + (size_t)g * D : nullptr);
+  auto channels = [&](int e, float (&out)[8]) {
+    load8(src + e, out);
+    if (bias != nullptr) {
+      float b[8];
+      load8(bias + e, b);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) out[i] += b[i];
+    }
+  };
+  // one over the root mean square of the head; every lane of the warp takes part (those without channels hold zeros)
+  auto inverse_rms = [&]() {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss = fmaf(x[i], x[i], ss);
+    for (int o = lph / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    return 1.f / sqrtf(ss / (float)D + eps);
+  };
+  auto weigh = [&](int e, float inv, float (&out)[8]) {
+    float wv[8];
+    load8(w + e, wv);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) out[i] *= inv * wv[i];
+  };
+  if (turns) channels(e0, x);
+  float inv = 1.f;
+  if (qw != nullptr) {
+    inv = inverse_rms();
+    if (turns) weigh(e0, inv, x);
+  }
+  if (cos_t != nullptr && turns && e0 < rot) {
+    const int half = rot / 2;
+    const bool low = e0 < half;
+    const int p0 = low ? e0 + half : e0 - half, f0 = low ? e0 : e0 - half;
+    float other[8], c[8], sn[8];
+    channels(p0, other);
+    if (qw != nullptr) weigh(p0, inv, other);
+    load8(cos_t + (size_t)n * half + f0, c);
+    load8(sin_t + (size_t)n * half + f0, sn);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] = low ? fmaf(x[i], c[i], -other[i] * sn[i]) : fmaf(x[i], c[i], other[i] * sn[i]);
+  }
+  if (unit) {
+    inv = inverse_rms();
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] *= inv;
+  }
+  if (turns) {
+    if (is_q) store8(q_out + ((size_t)n * H + head) * D + e0, x);
+    else store8(k_pool + (row + (long long)g * page_size) * D + e0, x);
+    return;
+  }
+  const int at = item - heads * lph;  // the values: 8 channels a thread
+  if (write && at >= 0 && at * 8 < G * V) {
+    const int c = at * 8, vg = c / V, j = c % V;
+    float y[8];
+    load8(v + (size_t)n * ldv + c, y);
+    if (vb != nullptr) {
+      float b[8];
+      load8(vb + c, b);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[i] += b[i];
+    }
+    store8(v_pool + (row + (long long)vg * page_size) * V + j, y);
+  }
+}
+
 // Scores of one key row against `heads` query rows in shared memory: the row is read once, 16 bytes at a time where
 // its size allows, and every head's sum is one ascending chain of fused multiply-adds.
 template <typename T>
@@ -282,6 +378,25 @@ AKAS_API int akas_qk_norm_store(const void* q, long long ldq, const void* k, lon
                                 const float* vb, int unit, cudaStream_t stream) {
   if (N <= 0) return 0;
   if (unit && (qw != nullptr || kw != nullptr)) return (int)cudaErrorInvalidValue;
+  if ((qw == nullptr) != (kw == nullptr)) return (int)cudaErrorInvalidValue;
+  const uintptr_t bases = (uintptr_t)q | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)qw | (uintptr_t)kw |
+                          (uintptr_t)cos_t | (uintptr_t)sin_t | (uintptr_t)qb | (uintptr_t)kb | (uintptr_t)vb |
+                          (write ? (uintptr_t)k | (uintptr_t)v : 0);
+  if (D % 8 == 0 && D <= 256 && V % 8 == 0 && (cos_t == nullptr || (!interleaved && rot % 16 == 0)) && bases % 16 == 0 && ldq % 8 == 0 &&
+      (!write || (ldk % 8 == 0 && ldv % 8 == 0))) {
+    int lph = 1;
+    while (lph < D / 8) lph *= 2;
+    const int threads = (write ? H + G : H) * lph + (write ? G * (V / 8) : 0);
+    const dim3 grid(N, (threads + 127) / 128);
+#define AKAS_STORE8(TI, T)                                                                                                    \
+  return launch_ordinary(qk_norm_store8_kernel<TI, T>, grid, dim3(128), 0, stream, (const TI*)q, ldq, (const TI*)k, ldk,      \
+                         (const TI*)v, ldv, qw, kw, eps, (T*)q_out, (T*)k_pool, (T*)v_pool, block_table, max_blocks,          \
+                         seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, qb, kb, vb, unit, lph)
+    if (dtype == AKAS_F32) AKAS_STORE8(float, float);
+    if (in_dtype == AKAS_F32) AKAS_STORE8(float, bf16);
+    AKAS_STORE8(bf16, bf16);
+#undef AKAS_STORE8
+  }
   if (cos_t != nullptr && (rot <= 0 || rot % 2 || rot > D)) return (int)cudaErrorInvalidValue;
   if (dtype == AKAS_F32 && in_dtype != AKAS_F32) return (int)cudaErrorInvalidValue;
   if (dtype == AKAS_F32)

@@ -249,8 +249,13 @@ grouped_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           for (int i = 0; i < 16; ++i) v[i] = __fdividef(v[i], 1.f + __expf(-v[i])) * u[i];  // the fast division: IEEE division cost more than the tile's loads
         }
         if (EPI == EPI_PLAIN) {
+          if (act == AKAS_PLAIN_RELU2) {
 #pragma unroll
-          for (int i = 0; i < 16; ++i) v[i] = plain_activation_fast(v[i], act);
+            for (int i = 0; i < 16; ++i) { const float r = fmaxf(v[i], 0.f); v[i] = r * r; }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) v[i] = plain_activation_fast(v[i], act);
+          }
         }
         const int col = n0 + c;
         if (row < M && col < out_cols) {

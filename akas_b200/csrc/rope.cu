@@ -100,14 +100,20 @@ __global__ void qk_norm_rope_store_kernel(T* __restrict__ qkv, T* __restrict__ q
   __syncwarp();
   T* dst = is_q ? q_out + (size_t)t * H * D + (size_t)head * D : src;
   const int half = rotary / 2;
+  auto turned = [&](int e) {
+    if (cos_t == nullptr || e >= rotary) return x[e];
+    const int f = e < half ? e : e - half;
+    const float c = cos_t[(size_t)t * half + f], s = sin_t[(size_t)t * half + f];
+    return e < half ? x[e] * c - x[e + half] * s : x[e - half] * s + x[e] * c;
+  };
+  float unit = 1.f;
+  if (zero_centered == AKAS_UNIT_BEHIND) {
+    float squares = 0.f;
+    for (int e = lane; e < D; e += 32) { const float v = turned(e); squares = fmaf(v, v, squares); }
+    unit = 1.f / sqrtf(warp_sum(squares) / (float)D + eps);
+  }
   for (int e = lane; e < D; e += 32) {
-    float v = x[e];
-    if (cos_t != nullptr && e < rotary) {
-      const int f = e < half ? e : e - half;
-      const float c = cos_t[(size_t)t * half + f], s = sin_t[(size_t)t * half + f];
-      v = e < half ? x[e] * c - x[e + half] * s : x[e - half] * s + x[e] * c;
-    }
-    const T o = from_f32<T>(v);
+    const T o = from_f32<T>(turned(e) * unit);
     dst[e] = o;
     if (page_row) page_row[e] = o;
   }
@@ -169,6 +175,7 @@ AKAS_API int akas_qk_norm_rope_store(void* qkv, void* q_out, const float* q_w, c
                                      const int* seq_of_token, const int* positions, int page_size, int N, int H,
                                      int KH, int D, int dtype, cudaStream_t stream) {
   if (D > 256 || D <= 0 || rotary > D || (rotary & 1)) return (int)cudaErrorInvalidValue;
+  if (zero_centered == AKAS_UNIT_BEHIND && (q_w != nullptr || k_w != nullptr)) return (int)cudaErrorInvalidValue;
   if (N <= 0) return 0;
   const bool wide = (D == 32 || D == 64 || D == 128 || D == 256) && rotary % 16 == 0 && (uintptr_t)qkv % 16 == 0 &&
                     (uintptr_t)q_out % 16 == 0 && (k_pool == nullptr || ((uintptr_t)k_pool % 16 == 0 && (uintptr_t)v_pool % 16 == 0)) &&

@@ -1099,9 +1099,20 @@ def rope_tables(positions, inv_freq, amplitude=1.0):
     return cos, sin
 
 
+_UNIT_BEHIND = 2
+
+
+def _norm_place(q_weight, zero_centered, unit) -> int:
+    """How the kernels between the qkv product and attention norm a head: 0 and 1 in front of the rotation with a weight
+    as it stands or one plus it (no weight: no norm), 2 behind the rotation without a weight (``unit``)."""
+    if unit and q_weight is not None:
+        raise ValueError("heads are normed in front of the rotation with a weight or behind it without")
+    return _UNIT_BEHIND if unit else int(bool(zero_centered))
+
+
 @_flushes
 def qk_norm_rope_store(qkv, heads, kv_heads, head_dim, q_weight, k_weight, eps, zero_centered, cos, sin,
-                       k_pool, v_pool, block_table, seq_of_token, positions, page_size):
+                       k_pool, v_pool, block_table, seq_of_token, positions, page_size, unit=False):
     n = qkv.shape[0]
     _dense(qkv, "qkv")
     if qkv.shape[1] != (heads + 2 * kv_heads) * head_dim:
@@ -1109,7 +1120,7 @@ def qk_norm_rope_store(qkv, heads, kv_heads, head_dim, q_weight, k_weight, eps, 
     q = torch.empty((n, heads * head_dim), dtype=qkv.dtype, device=qkv.device)
     rotary = 2 * cos.shape[1] if cos is not None else 0
     _check(_fn("rope", "akas_qk_norm_rope_store")(
-        _ptr(qkv), _ptr(q), _ptr(q_weight), _ptr(k_weight), float(eps), int(bool(zero_centered)), _ptr(cos), _ptr(sin),
+        _ptr(qkv), _ptr(q), _ptr(q_weight), _ptr(k_weight), float(eps), _norm_place(q_weight, zero_centered, unit), _ptr(cos), _ptr(sin),
         rotary, _ptr(k_pool), _ptr(v_pool), _ptr(block_table), block_table.shape[1], _ptr(seq_of_token),
         _ptr(positions), page_size, n, heads, kv_heads, head_dim, _code(qkv), _stream()), "qk_norm_rope_store")
     return q
@@ -1263,7 +1274,7 @@ fused_qkv_attention = os.environ.get("AKAS_B200_FUSED_QKV_ATTENTION", "1") != "0
 
 @_flushes
 def qkv_decode_attention(qkv, heads, kv_heads, head_dim, q_weight, k_weight, eps, zero_centered, cos, sin, k_pool, v_pool,
-                         block_table, seq_of_token, positions, scale, window, page_size, ctx, write=True):
+                         block_table, seq_of_token, positions, scale, window, page_size, ctx, write=True, unit=False):
     """``paged_attention(qk_norm_rope_store(qkv, ...), ...)`` for a decode step (every token the single token of its
     request) in one launch, or None where the fused kernel does not take the sizes or the dtype (the caller then runs
     the two by themselves). With ``write=False`` the pages are read as they are and nothing is written."""
@@ -1285,7 +1296,7 @@ def qkv_decode_attention(qkv, heads, kv_heads, head_dim, q_weight, k_weight, eps
     if splits > 1:
         part_o = torch.empty((n, heads, splits, head_dim), dtype=torch.float32, device=qkv.device)
         part_ml = torch.empty((n, heads, splits, 2), dtype=torch.float32, device=qkv.device)
-    prep = (_ptr(qkv), _ptr(q_weight), _ptr(k_weight), float(eps), int(bool(zero_centered)), _ptr(cos), _ptr(sin), rotary,
+    prep = (_ptr(qkv), _ptr(q_weight), _ptr(k_weight), float(eps), _norm_place(q_weight, zero_centered, unit), _ptr(cos), _ptr(sin), rotary,
             int(bool(write)), _ptr(k_pool), _ptr(v_pool), k_pool.shape[0], _ptr(block_table), block_table.shape[1],
             _ptr(seq_of_token), _ptr(positions), _ptr(out), _ptr(part_o), _ptr(part_ml), float(scale), win, page_size, n,
             heads, kv_heads, head_dim, splits, _stream())

@@ -139,8 +139,9 @@ def kv_store(k, v, k_pool, v_pool, block_table, seq_of_token, positions, page_si
 
 
 def qk_norm_rope_store(qkv, heads, kv_heads, head_dim, q_weight, k_weight, eps, zero_centered, cos, sin,
-                       k_pool, v_pool, block_table, seq_of_token, positions, page_size):
-    """Per-head RMSNorm of q and k, rotation of both, k (in place in ``qkv``) and v into the pages; returns q."""
+                       k_pool, v_pool, block_table, seq_of_token, positions, page_size, unit=False):
+    """Per-head RMSNorm of q and k, rotation of both, k (in place in ``qkv``) and v into the pages; returns q. ``unit``:
+    no norm in front of the rotation; behind it every head over sqrt(mean of its squares + eps), without a weight."""
     n = qkv.shape[0]
     d = head_dim
     q = qkv[:, : heads * d].reshape(n, heads, d).to(torch.float32)
@@ -157,6 +158,8 @@ def qk_norm_rope_store(qkv, heads, kv_heads, head_dim, q_weight, k_weight, eps, 
             return torch.cat((left * c - right * s, left * s + right * c, rest), dim=-1)
 
         q, k = rotate(q), rotate(k)
+    if unit:
+        q, k = (x * torch.rsqrt((x * x).mean(dim=-1, keepdim=True) + eps) for x in (q, k))
     qkv[:, heads * d : (heads + kv_heads) * d] = k.reshape(n, kv_heads * d).to(qkv.dtype)
     if k_pool is not None:
         kv_store(qkv[:, heads * d : (heads + kv_heads) * d], qkv[:, (heads + kv_heads) * d :], k_pool, v_pool,

@@ -2,8 +2,9 @@
 
 In order (src/akas/models/lfm2/_composition.py:234-307 in kreasof-ai/akas): one
 product for q, k and v (their three matrices are stacked at load); RMSNorm of each
-head of q and k over head_dim, then the position encoding of q and k, and the
-write of k and v into the pages at each token's absolute position (one kernel);
+head of q and k over head_dim, then the position encoding of q and k (or, where the
+spec says so, the position encoding first and then the division of each head by its
+root mean square, without a weight), and the write of k and v into the pages at each token's absolute position (one kernel);
 attention of every query over the keys of its own request up to its own position,
 read from the pages, so a portion of a prompt attends to what earlier steps left
 and to itself; the output product, added to the residual.
@@ -11,8 +12,7 @@ and to itself; the output product, added to the residual.
 A layer whose spec asks for more than that (value heads of another size than the keys', a capped score, a
 logarithmic distance penalty, first tokens kept behind the window, a sink in the softmax's denominator (exp(0) or a
 learned logit per head), a gate per head on the output, values that are the keys as projected, rotary pairs of
-neighbouring channels, biases on q, k and v, heads of q and k divided by their root mean square after the position
-encoding, no keys and values of its own but another layer's cache) runs the same
+neighbouring channels, biases on q, k and v, no keys and values of its own but another layer's cache) runs the same
 steps on the general kernels: one product for q, k, v and the gate's
 logits, QK-norm, rotation and page write (``ops.qk_norm_store``), attention with the options as arguments
 (``ops.attention_general``), the output product. ``core`` is that sequence without the two products, for a mixer
@@ -67,6 +67,8 @@ class Attention(Mixer):
         self.scale = s.scale if s.scale is not None else s.head_dim ** -0.5
         if self.general and self.position is not None and not hasattr(self.position, "tables"):
             raise ValueError("the general attention kernels take a position encoding by rotary tables only")
+        if self.unit_eps is not None and self.position is not None and not hasattr(self.position, "tables"):
+            raise ValueError("heads are normed behind a position encoding by rotary tables only")
         self.w_qkv = None
         self.w_out = None
         self.r1 = self.r2 = self.sinks = self.bias = None
@@ -214,14 +216,17 @@ class Attention(Mixer):
         if self.position is not None and fused:
             cos, sin = self.position.tables(ctx)
         norm = self.q_norm.spec if self.q_norm is not None else None
+        eps, unit = norm.eps if norm else 0.0, {}
+        if self.unit_eps is not None:
+            eps, unit = self.unit_eps, dict(unit=True)
         if fused and ctx.decode_only and hasattr(ops, "qkv_decode_attention"):
             # a decode step: everything between the qkv product and the output product as one kernel, where there is one
             out = ops.qkv_decode_attention(
                 qkv, s.num_heads, s.num_kv_heads, s.head_dim,
                 self.q_norm.weight if norm else None, self.k_norm.weight if norm else None,
-                norm.eps if norm else 0.0, bool(norm and norm.zero_centered), cos, sin, cache.k, cache.v,
+                eps, bool(norm and norm.zero_centered), cos, sin, cache.k, cache.v,
                 ctx.block_table(cache.group), ctx.seq_of_token, ctx.positions, self.scale, s.window, cache.page_size,
-                ctx, write=write,
+                ctx, write=write, **unit,
             )
             if out is not None:
                 return project(self.rt, out, self.w_out, residual=residual)
@@ -229,9 +234,9 @@ class Attention(Mixer):
         q = ops.qk_norm_rope_store(
             qkv, s.num_heads, s.num_kv_heads, s.head_dim,
             self.q_norm.weight if norm else None, self.k_norm.weight if norm else None,
-            norm.eps if norm else 0.0, bool(norm and norm.zero_centered), cos, sin,
+            eps, bool(norm and norm.zero_centered), cos, sin,
             cache.k if store else None, cache.v if store else None,
-            ctx.block_table(cache.group), ctx.seq_of_token, ctx.positions, cache.page_size,
+            ctx.block_table(cache.group), ctx.seq_of_token, ctx.positions, cache.page_size, **unit,
         )
         if not fused:
             # A position encoding without rotary tables rewrites q and k itself; k and v go to the pages after it.

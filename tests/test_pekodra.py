@@ -20,7 +20,7 @@ import torch
 import plain_pekodra as plain
 import traces
 
-from tiny_pekodra import (ATT, ATT_BARE, ATT_FULL, ATT_MID, ATT_ODD, ATT_SELF, BLEND, CONFIGS, LENGTHS, PAGE, TOL, attn, dense, layer,
+from tiny_pekodra import (ATT, ATT_BARE, ATT_EVEN, ATT_EVEN32, ATT_EVEN64, ATT_FULL, ATT_ODD, ATT_SELF, BLEND, CONFIGS, LENGTHS, PAGE, TOL, attn, dense, layer,
                           make_folder, model, moe, plant, prompts)
 
 ROOT = Path(__file__).resolve().parent.parent
@@ -122,6 +122,9 @@ def test_config_round_trip_registry_and_inventory(tmp_path):
     assert second.ffn.kind == "gated_mlp" and second.ffn.activation == "gelu_tanh" and second.ffn.bias and second.ffn.intermediate_size == 48
     assert spec.head_name == "head" and spec.logit_scale == 0.7 and spec.embedding_multiplier == 3.0
     assert set(kernel_kinds(spec)) == {"attention_general", "rope", "moe"}
+    # values of the keys' size, at sizes that the kernels for plain attention take: those, whatever the norm's place
+    even = config_from_dict(CONFIGS["even"]).model_spec()
+    assert not any(l.mixer.general for l in even.layers) and set(kernel_kinds(even)) == {"attention", "moe"}
     assert config_from_dict(CONFIGS["alone"]).loop is None
     folder, _ = make_folder(CONFIGS["odd"], seed=1, folder=tmp_path / "m")
     assert load_config(folder) == config_from_dict(CONFIGS["odd"])
@@ -232,7 +235,7 @@ def test_unit_heads_behind_the_rotation():
     assert torch.allclose((want * want).mean(-1), torch.ones(37, 4, dtype=plain.F), atol=1e-3)
 
 
-@pytest.mark.parametrize("mixer", [ATT, ATT_FULL, ATT_ODD, ATT_SELF, ATT_BARE])
+@pytest.mark.parametrize("mixer", [ATT, ATT_FULL, ATT_ODD, ATT_SELF, ATT_BARE, ATT_EVEN, ATT_EVEN32, ATT_EVEN64])
 def test_attention_alone(mixer, tmp_path):
     one_mechanism(model(48, 60, [layer(mixer, None)]), tmp_path)
 
@@ -326,16 +329,19 @@ def test_the_loop_and_the_embedding_that_joins(tmp_path):
 
 
 WINDOW = 130
+KINDS = {"general": (dict(ATT, mask=dict(size=WINDOW), scale=1.0), 8),
+         "plain": (dict(ATT_EVEN64, mask=dict(size=WINDOW), scale=0.3), 64), "plain, small pages": (dict(ATT_EVEN, mask=dict(size=WINDOW), scale=1.5), 8)}
 
 
-def seen_case(device, dtype, ops, tmp_path, decode):
+def seen_case(device, dtype, ops, tmp_path, decode, kind):
     """One layer: the logits at position i change with the token at position j iff i - WINDOW < j <= i: just inside and
     just outside the window, keys at page borders, next to the query, the query itself; later tokens never; with the
     query in a prompt's portion or decoded alone."""
     from akas_b200.engine.batch import StepEntry
 
     i = 290
-    config = model(48, 120, [layer(dict(ATT, mask=dict(size=WINDOW), scale=1.0), None)])
+    mixer, page = KINDS[kind]
+    config = model(48, 120, [layer(mixer, None)])
     folder, _ = make_folder(config, seed=44, folder=tmp_path / "edge")
     w = plant(folder, config, key_token=119, query_token=118)  # token 119 at position j is felt by token 118 at position i
     edge = i - WINDOW + 1
@@ -345,7 +351,7 @@ def seen_case(device, dtype, ops, tmp_path, decode):
     base[i] = 118
 
     def logits_at_i(tokens):
-        runner = runner_for(folder, dtype, device, 8, 320, ops)
+        runner = runner_for(folder, dtype, device, page, 320, ops)
         if decode:
             runner.step([StepEntry("a", tokens[:i], ())])
             out = runner.step([StepEntry("a", tokens[i:i + 1], (0,))])
@@ -369,27 +375,30 @@ def seen_case(device, dtype, ops, tmp_path, decode):
             assert np.abs(got - want).max() <= TOL[dtype] * np.abs(want).max()
 
 
+@pytest.mark.parametrize("kind", list(KINDS))
 @pytest.mark.parametrize("decode", [False, True])
-def test_what_a_position_sees_on_the_plain_operations(decode, tmp_path):
+def test_what_a_position_sees_on_the_plain_operations(decode, kind, tmp_path):
     from akas_b200.ops import reference
 
-    seen_case("cpu", "float32", reference, tmp_path, decode)
+    seen_case("cpu", "float32", reference, tmp_path, decode, kind)
 
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("kind", list(KINDS))
 @pytest.mark.parametrize("decode", [False, True])
-def test_what_a_position_sees_on_the_kernels(decode, dtype, tmp_path):
-    seen_case("cuda:0", dtype, None, tmp_path, decode)
+def test_what_a_position_sees_on_the_kernels(decode, dtype, kind, tmp_path):
+    seen_case("cuda:0", dtype, None, tmp_path, decode, kind)
 
 
-def far_key_case(device, dtype, ops, tmp_path):
+def far_key_case(device, dtype, ops, tmp_path, kind):
     """One key far back among hundreds is made to stand out, as the oldest one that the window still holds: the last
     position's attention must find it through scattered pages, in a portion and decoded alone, in every pass of a looped
     layer (each has its own pages); one position further back it must be gone."""
     from akas_b200.engine.batch import StepEntry
 
-    config = model(48, 120, [layer(dict(ATT, mask=dict(size=497), scale=1.0), None)], loop=(0, 1, 2))
+    mixer, page = KINDS[kind]
+    config = model(48, 120, [layer(dict(mixer, mask=dict(size=497)), None)], loop=(0, 1, 2))
     folder, _ = make_folder(config, seed=47, folder=tmp_path / "far")
     w = plant(folder, config, key_token=119, query_token=118)
     toks = prompts(118, [500], seed=2)[0]
@@ -404,7 +413,8 @@ def far_key_case(device, dtype, ops, tmp_path):
     assert felt > 0.1 * np.abs(want).max() and np.abs(past - want).max() > 0.1 * np.abs(want).max(), "the far key does not stand out"
     for tokens, expected in ((toks, want), (moved, past)):
         for cuts in ([500], [499, 1], [130, 70, 2, 290, 8]):
-            runner = runner_for(folder, dtype, device, 16, 576, ops, context=512)
+            runner = runner_for(folder, dtype, device, 2 * page, 640, ops, context=512) if page < 64 else \
+                runner_for(folder, dtype, device, page, 640, ops, context=512)
             runner.admit("other")  # the request's pages are not the pool's first
             runner.cache.reserve("other", 40)
             at = 0
@@ -415,16 +425,18 @@ def far_key_case(device, dtype, ops, tmp_path):
             assert np.abs(got - expected).max() <= TOL[dtype] * np.abs(expected).max(), cuts
 
 
-def test_a_far_key_is_found_on_the_plain_operations(tmp_path):
+@pytest.mark.parametrize("kind", list(KINDS))
+def test_a_far_key_is_found_on_the_plain_operations(kind, tmp_path):
     from akas_b200.ops import reference
 
-    far_key_case("cpu", "float32", reference, tmp_path)
+    far_key_case("cpu", "float32", reference, tmp_path, kind)
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("kind", list(KINDS))
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-def test_a_far_key_is_found_on_the_kernels(dtype, tmp_path):
-    far_key_case("cuda:0", dtype, None, tmp_path)
+def test_a_far_key_is_found_on_the_kernels(dtype, kind, tmp_path):
+    far_key_case("cuda:0", dtype, None, tmp_path, kind)
 
 
 def test_freed_pages_are_used_again_and_not_read(tmp_path):
@@ -641,8 +653,75 @@ def test_unit_heads_behind_the_rotation_kernel(heads, kv_heads, dim, vdim, dims,
     for want, got in zip(results[:2], results[2:]):
         for a, b, what in zip(got, want, ("queries", "keys", "values")):
             _close(a, b, tol, what)
+    # the same kernel with a weighted norm in front of the rotation, and with biases on float32 products
+    g = torch.Generator().manual_seed(1)
+    weights = [torch.rand(dim, generator=g) + 0.5 for _ in range(2)]
+    biases = [torch.randn(width, generator=g) for width in (heads * dim, kv_heads * dim, kv_heads * vdim)]
+    for weighted in (False, True):
+        pair = []
+        for ops, device in ((reference, "cpu"), (cuda, "cuda")):
+            if dims:
+                tables = dict(cos=cos.to(device), sin=sin.to(device))
+            pools = [torch.zeros(pages, kv_heads, page, width, dtype=dtype, device=device) for width in (dim, vdim)]
+            w = [x.to(device) if weighted else None for x in weights]
+            out = ops.qk_norm_store(q.float().to(device), k.float().to(device), v.float().to(device), heads, kv_heads, dim, vdim, *w, 1e-4,
+                                    *pools, table.to(device), seq.to(device), pos.to(device), page, **tables,
+                                    **dict(zip(("q_bias", "k_bias", "v_bias"), (b.to(device) for b in biases))))
+            pair.append((out, *pools))
+        for a, b, what in zip(pair[1], pair[0], ("queries", "keys", "values")):
+            _close(a, b, tol, f"{what}, biases, weights {weighted}")
     want = plain.rms(plain.rotate(q.double().reshape(-1, heads, dim), rot) if dims else q.double().reshape(-1, heads, dim), 1e-4)
     _close(results[2][0].reshape(-1, heads, dim), want, tol, "queries against the equations")
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("heads,kv_heads,dim,dims,page", [(6, 2, 16, 12, 8), (4, 1, 32, 32, 16), (8, 2, 64, 32, 64), (5, 5, 64, 64, 64),
+                                                         (2, 1, 128, 64, 64), (3, 3, 48, 0, 8), (2, 1, 256, 16, 32)])
+def test_unit_heads_from_the_stacked_product(heads, kv_heads, dim, dims, page, dtype):
+    """The kernel between the stacked q, k, v product and plain attention, and (head size 64, bfloat16) the decode kernel
+    that does it on its way: heads divided by their root mean square behind the rotation."""
+    from akas_b200.ops import cuda, reference
+
+    cuda.require(["rope", "attention"] + (["attention_decode"] if dtype == torch.bfloat16 else []))
+    rot = dict(base=300.0, dims=dims, scaling=BLEND)
+    q, k, v, table, seq, pos, pages = _unit_case(heads, kv_heads, dim, dim, rot, page)
+    qkv = torch.cat([q, k, v], dim=1).to(dtype)
+    tables = (None, None)
+    if dims:
+        freq, amp = plain.rates(rot)
+        tables = reference.rope_tables(pos, torch.tensor(freq, dtype=torch.float64), amp)
+    results = []
+    for ops, device in ((reference, "cpu"), (cuda, "cuda")):
+        pools = [torch.zeros(pages, kv_heads, page, dim, dtype=dtype, device=device) for _ in range(2)]
+        at = [t.to(device) if t is not None else None for t in tables]
+        out = ops.qk_norm_rope_store(qkv.clone().to(device), heads, kv_heads, dim, None, None, 1e-4, False, *at, *pools, table.to(device),
+                                     seq.to(device), pos.to(device), page, unit=True)
+        results.append((out, *pools))
+    tol = 2e-6 if dtype == torch.float32 else 8e-3
+    for a, b, what in zip(results[1], results[0], ("queries", "keys", "values")):
+        _close(a, b, tol, what)
+    turned = qkv[:, : heads * dim].double().reshape(-1, heads, dim)
+    _close(results[1][0].reshape(-1, heads, dim), plain.rms(plain.rotate(turned, rot) if dims else turned, 1e-4), tol, "against the equations")
+    if dtype == torch.bfloat16 and dim == 64:
+        # the last token decoded: its page row is not there yet
+        class Ctx:
+            max_context = 64
+            query_lens = (1,)
+
+        n = qkv.shape[0]
+        want = reference.paged_attention(results[0][0][n - 1:], *results[0][1:], table, seq[n - 1:], pos[n - 1:], 0.2, 21, page)
+        pools = [p.clone() for p in results[1][1:]]
+        where = int(table[0, (n - 1) // page]), (n - 1) % page
+        for p in pools:
+            p[where[0], :, where[1]] = 0.0
+        one = [t[n - 1:].cuda().contiguous() if t is not None else None for t in tables]
+        got = cuda.qkv_decode_attention(qkv[n - 1:].cuda().contiguous(), heads, kv_heads, dim, None, None, 1e-4, False, *one, *pools, table.cuda(),
+                                        seq[n - 1:].cuda(), pos[n - 1:].cuda(), 0.2, 21, page, Ctx, unit=True)
+        assert got is not None
+        _close(got, want, 1.5e-2, "decode attention from the product")
+        _close(pools[0], results[1][1], 8e-3, "the key written on the way")
+        assert torch.equal(pools[1], results[1][2])
 
 
 @pytest.mark.gpu

@@ -29,6 +29,11 @@ ATT_ODD = attn(3, 1, 20, 28, 33, 0.45, 1000000.0, 6, dict(factor=1.5, original=1
 ATT_SELF = attn(5, 5, 12, 10, 1, 0.7, 500.0, 4)     # every position sees itself only
 ATT_BARE = attn(12, 2, 8, 8, 1000, 0.9, 100.0, 0)  # no rotation; a window longer than any prompt here
 ATT_MID = attn(8, 2, 64, 48, 90, 0.2, 10000.0, 32, dict(factor=8.0, original=512, fast=16.0, slow=2.0))
+# values of the keys' size, at sizes that the kernels for plain attention take
+ATT_EVEN = attn(6, 2, 16, 16, 27, 0.6, 10000.0, 12, dict(factor=2.0, original=200, fast=8.0, slow=1.0))
+ATT_EVEN32 = attn(4, 1, 32, 32, 40, 0.3, 300.0, 32, BLEND)
+ATT_EVEN64 = attn(8, 2, 64, 64, 75, 0.2, 10000.0, 32, dict(factor=8.0, original=512, fast=16.0, slow=2.0))
+ATT_EVEN128 = attn(2, 2, 128, 128, 66, 0.1, 500000.0, 128, dict(factor=5.0, original=300, fast=16.0, slow=1.0))
 ATT_MID2 = attn(4, 4, 32, 64, 64, 0.35, 500000.0, 32, dict(factor=3.0, original=128, fast=32.0, slow=1.0))
 
 
@@ -70,13 +75,15 @@ CONFIGS = {
     "ragged": model(50, 77, [layer(ATT_BARE, moe(10, 3, 2, shared=6)), layer(ATT_ODD, dense(14)), layer(ATT_SELF, None)], loop=(1, 2, 1),
                     eps=1e-3, logit_scale=-2.2, embedding_scale=1.0),
     "alone": model(48, 120, [layer(ATT, dense(24)), layer(ATT_ODD, moe(24, 4, 1, shared=24))], embedding_scale=11.5),  # no loop at all
+    "even": model(64, 110, [layer(ATT_EVEN, dense(32)), layer(ATT_EVEN64, moe(32, 4, 2, shared=24)), layer(ATT_EVEN128, None),
+                            layer(ATT_EVEN32, dense(48))], loop=(1, 3, 2), embedding_scale=1.5),
     # sizes that the tensor-core kernels take, with a looped last layer
     "mid": model(128, 300, [layer(ATT_MID, dense(192)), layer(ATT_MID2, moe(64, 8, 2, shared=64)), layer(ATT_MID, moe(136, 4, 1, shared=192))],
                  loop=(2, 3, 2), eps=1e-6, logit_scale=0.5, embedding_scale=2.0),
 }
-PAGE = {"mix": 8, "odd": 16, "ragged": 32, "alone": 64, "mid": 64}
+PAGE = {"mix": 8, "odd": 16, "ragged": 32, "alone": 64, "even": 64, "mid": 64}
 LENGTHS = {"mix": [1, 45, 2, 97, 33, 130, 64], "odd": [70, 3, 41, 100], "ragged": [75, 2, 140], "alone": [90, 1, 150],
-           "mid": [200, 129, 64]}
+           "even": [150, 40, 2, 210], "mid": [200, 129, 64]}
 LOUD = 1.0  # how far the directions that the routers read stand out of the rest of an embedding
 TOL = {"float32": 3e-5, "bfloat16": 2e-2}  # largest |difference| over largest |reference logit|
 
