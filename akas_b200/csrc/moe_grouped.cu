@@ -10,6 +10,8 @@
 //   grouped product (the persistent, TMA-fed, tcgen05 kernel of gemm_tcgen05.cu with an expert per tile): B tiles
 //                come from the stacked matrices [experts * rows, K] at the tile's expert;
 //                  SWIGLU: act[row, F] = silu(gate) * up, bfloat16;   F32: y[row, C] = act . W_down^T, float32;
+//                (a warp's 32 rows of 32 or 64 channels go to a swizzled staging tile, two per warp in turn, and by TMA to
+//                memory: rows written 32 bytes at a time by their lanes cost more than the products)
 //                  PLAIN: act[row, F] = an activation without a gate (ungated experts, matrices [experts * F, K]), bfloat16.
 //   moe_combine  out[n] = sum_k weight[n, k] * (y[row of pair (n, k)], or h[n] for an identity expert), in the
 //                order of the choice, float32; or, given the residual stream x, x += mult * (ls_a * a + ls_b * that sum).
@@ -26,6 +28,7 @@ namespace {
 
 constexpr int BM = 128, STAGES = 4;
 constexpr int THREADS = 192;
+constexpr int STAGING = 4096;  // bytes of one staging tile of the read-out: 32 rows x 128 bytes (SWIGLU: 64)
 enum { EPI_F32 = 1, EPI_SWIGLU = 2, EPI_PLAIN = 4 };
 
 __device__ int g_grouped_status = 0;  // 0, or which bounded wait ran out last (1 producer, 2 tensor cores, 3 epilogue)
@@ -134,7 +137,7 @@ __global__ void moe_combine_kernel(const bf16* __restrict__ h, long long ldh, co
 template <int BN, int EPI>
 __global__ void __launch_bounds__(THREADS)
 grouped_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-               void* __restrict__ y_, const int* __restrict__ tile_expert, const int* __restrict__ plan, int N, int K, int F,
+               const __grid_constant__ CUtensorMap map_y, const int* __restrict__ tile_expert, const int* __restrict__ plan, int N, int K, int F,
                int act) {
   // A tile's B rows are those of its expert in the stacked matrix [experts * N, K]; M is what the plan kernel counted.
   // N: channels of the product (for SWIGLU the stacked height 2F); a tile covers BN of them (SWIGLU: BN/2 gate
@@ -149,7 +152,6 @@ grouped_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int out_cols = EPI == EPI_SWIGLU ? F : N;
   const int tiles_m = plan[0], tiles_n = (out_cols + TILE_N - 1) / TILE_N;
-  const int M = tiles_m * BM;
   const int tiles = tiles_m * tiles_n, k_blocks = (K + BK - 1) / BK;
 
   if (tid == 0) {
@@ -229,62 +231,76 @@ grouped_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
   } else {
     // ------------------------------------------------------------------ epilogue: warps 2..5
     const int sub = warp & 3;  // the tensor-memory sub-partition (32 lanes) this warp may read
-    unsigned t = 0;
+    unsigned char* staging = smem + (size_t)STAGES * STAGE_BYTES + (size_t)sub * 2 * STAGING;
+    unsigned t = 0, stores = 0;
     for (int tile = blockIdx.x; tile < tiles; tile += gridDim.x, ++t) {
       const unsigned acc = t & 1;
       const int m0 = (tile / tiles_n) * BM, n0 = (tile % tiles_n) * TILE_N;
       wait_for(&acc_full[acc], (t >> 1) & 1, 3);
       if (*(volatile int*)&abort_s) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const int row = m0 + sub * 32 + lane;
+      const int row0 = m0 + sub * 32;  // this warp's 32 rows; lane l holds row0 + l
       const unsigned taddr = tmem_base + acc * BN + ((unsigned)(sub * 32) << 16);
+      constexpr int COLS = EPI == EPI_PLAIN ? 64 : 32;  // output columns per staging tile
 #pragma unroll 1
-      for (int c = 0; c < TILE_N; c += 16) {
-        float v[16];
-        tmem_load16(taddr + c, v);
-        if (EPI == EPI_SWIGLU) {
-          float u[16];
-          tmem_load16(taddr + BN / 2 + c, u);
+      for (int c = 0; c < TILE_N; c += COLS, ++stores) {
+        if (n0 + c >= out_cols) break;
+        unsigned char* buf = staging + (size_t)(stores & 1) * STAGING;
+        if (lane == 0) bulk_wait_read<1>();  // the store before last has read this tile
+        __syncwarp();
+        float v[32], u[32];
+        tmem_load32(taddr + c, v);
+        if (EPI == EPI_F32) {
+          // row `lane` of 128 bytes, its 16-byte units XORed with the row's number within eight (the 128-byte swizzle)
 #pragma unroll
-          for (int i = 0; i < 16; ++i) v[i] = __fdividef(v[i], 1.f + __expf(-v[i])) * u[i];  // the fast division: IEEE division cost more than the tile's loads
-        }
-        if (EPI == EPI_PLAIN) {
+          for (int j = 0; j < 8; ++j)
+            *reinterpret_cast<float4*>(buf + lane * 128 + ((j ^ (lane & 7)) << 4)) =
+                make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
+        } else if (EPI == EPI_PLAIN) {
+          tmem_load32(taddr + c + 32, u);
           if (act == AKAS_PLAIN_RELU2) {
 #pragma unroll
-            for (int i = 0; i < 16; ++i) { const float r = fmaxf(v[i], 0.f); v[i] = r * r; }
-          } else {
-#pragma unroll
-            for (int i = 0; i < 16; ++i) v[i] = plain_activation_fast(v[i], act);
-          }
-        }
-        const int col = n0 + c;
-        if (row < M && col < out_cols) {
-          if (EPI == EPI_F32) {
-            float* dst = (float*)y_ + (size_t)row * out_cols + col;
-            if (col + 16 <= out_cols && out_cols % 4 == 0) {
-#pragma unroll
-              for (int i = 0; i < 16; i += 4) *reinterpret_cast<float4*>(dst + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
-            } else {
-              for (int i = 0; i < 16 && col + i < out_cols; ++i) dst[i] = v[i];
+            for (int i = 0; i < 32; ++i) {
+              v[i] = fmaxf(v[i], 0.f) * fmaxf(v[i], 0.f);
+              u[i] = fmaxf(u[i], 0.f) * fmaxf(u[i], 0.f);
             }
           } else {
-            bf16* dst = (bf16*)y_ + (size_t)row * out_cols + col;
-            if (col + 16 <= out_cols && out_cols % 8 == 0) {
-              float lo[8], hi[8];
 #pragma unroll
-              for (int i = 0; i < 8; ++i) { lo[i] = v[i]; hi[i] = v[8 + i]; }
-              store_vec(dst, lo);
-              store_vec(dst + 8, hi);
-            } else {
-              for (int i = 0; i < 16 && col + i < out_cols; ++i) dst[i] = __float2bfloat16_rn(v[i]);
-            }
+            for (int i = 0; i < 32; ++i) { v[i] = plain_activation_fast(v[i], act); u[i] = plain_activation_fast(u[i], act); }
+          }
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            uint4 o, p;
+            o.x = pack2(v[8 * j], v[8 * j + 1]); o.y = pack2(v[8 * j + 2], v[8 * j + 3]);
+            o.z = pack2(v[8 * j + 4], v[8 * j + 5]); o.w = pack2(v[8 * j + 6], v[8 * j + 7]);
+            p.x = pack2(u[8 * j], u[8 * j + 1]); p.y = pack2(u[8 * j + 2], u[8 * j + 3]);
+            p.z = pack2(u[8 * j + 4], u[8 * j + 5]); p.w = pack2(u[8 * j + 6], u[8 * j + 7]);
+            *reinterpret_cast<uint4*>(buf + lane * 128 + ((j ^ (lane & 7)) << 4)) = o;
+            *reinterpret_cast<uint4*>(buf + lane * 128 + (((j + 4) ^ (lane & 7)) << 4)) = p;
+          }
+        } else {
+          tmem_load32(taddr + BN / 2 + c, u);
+#pragma unroll
+          for (int i = 0; i < 32; ++i) v[i] = __fdividef(v[i], 1.f + __expf(-v[i])) * u[i];  // the fast division: IEEE division cost more than the tile's loads
+          // row `lane` of 64 bytes, its 16-byte units XORed with bits 7-8 of the address (the 64-byte swizzle)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            uint4 o;
+            o.x = pack2(v[8 * j], v[8 * j + 1]); o.y = pack2(v[8 * j + 2], v[8 * j + 3]);
+            o.z = pack2(v[8 * j + 4], v[8 * j + 5]); o.w = pack2(v[8 * j + 6], v[8 * j + 7]);
+            *reinterpret_cast<uint4*>(buf + lane * 64 + ((j ^ ((lane >> 1) & 3)) << 4)) = o;
           }
         }
+        fence_async_smem();
+        __syncwarp();
+        if (lane == 0) { tma_store_2d(&map_y, buf, n0 + c, row0); bulk_commit(); }
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       __syncwarp();
       if (lane == 0) mbar_arrive(&acc_empty[acc]);
     }
+    if (lane == 0) bulk_wait_all();  // what this warp handed to TMA has been written before the block may leave
+    __syncwarp();
   }
 
   // wind down: everyone meets, then the allocating warp frees tensor memory
@@ -304,7 +320,7 @@ grouped_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
 template <int BN, int EPI>
 int launch(const void* x, const void* w, void* y, const int* tile_expert, const int* plan, int rows_cap, int experts, int N,
            int K, int act, cudaStream_t stream) {
-  constexpr int smem = STAGES * (BM * BK * 2 + BN * BK * 2) + 1024;
+  constexpr int smem = STAGES * (BM * BK * 2 + BN * BK * 2) + 8 * STAGING + 1024;
   static int sms_of[64] = {};
   int device = 0;
   if (cudaGetDevice(&device) != cudaSuccess || device < 0 || device >= 64) return (int)cudaErrorInvalidDevice;
@@ -315,15 +331,17 @@ int launch(const void* x, const void* w, void* y, const int* tile_expert, const 
   }
   const int sms = sms_of[device];
   const int F = N / 2;
-  CUtensorMap map_x, map_w;
+  CUtensorMap map_x, map_w, map_y;
   int err = cached_map(&map_x, x, rows_cap, K, BM, false);
   if (err) return err;
   err = cached_map(&map_w, w, experts * N, K, EPI == EPI_SWIGLU ? BN / 2 : BN, true);
   if (err) return err;
   const int out_cols = EPI == EPI_SWIGLU ? F : N, tile_n = EPI == EPI_SWIGLU ? BN / 2 : BN;
+  err = EPI == EPI_F32 ? make_store_map(&map_y, y, rows_cap, out_cols, 4, 32) : make_store_map(&map_y, y, rows_cap, out_cols, 2, EPI == EPI_PLAIN ? 64 : 32);
+  if (err) return err;
   const long long most = (long long)(rows_cap / BM) * ((out_cols + tile_n - 1) / tile_n);
   const int grid = most < sms ? (int)most : sms;
-  grouped_kernel<BN, EPI><<<grid, THREADS, smem, stream>>>(map_x, map_w, y, tile_expert, plan, N, K, F, act);
+  grouped_kernel<BN, EPI><<<grid, THREADS, smem, stream>>>(map_x, map_w, map_y, tile_expert, plan, N, K, F, act);
   return launch_status();
 }
 
@@ -365,7 +383,7 @@ AKAS_API int akas_moe_grouped_gemm(const void* x, const void* w, void* y, const 
     return N <= 128 ? launch<128, EPI_PLAIN>(x, w, y, tile_expert, plan, rows_cap, experts, N, K, act, stream)
                     : launch<256, EPI_PLAIN>(x, w, y, tile_expert, plan, rows_cap, experts, N, K, act, stream);
   }
-  if (epilogue != EPI_F32) return (int)cudaErrorInvalidValue;
+  if (epilogue != EPI_F32 || N % 4) return (int)cudaErrorInvalidValue;
   // (128 x 128 tiles for steps whose 128 x 256 tiles would leave SMs without one were measured and dropped: the down
   // product of 64 tokens over 14 experts took 48 us against 43 us)
   return N <= 128 ? launch<128, EPI_F32>(x, w, y, tile_expert, plan, rows_cap, experts, N, K, 0, stream)
