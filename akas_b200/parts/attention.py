@@ -208,8 +208,6 @@ class Attention(Mixer):
         s, ops = self.spec, self.rt.ops
         if self.general:
             return self._forward_general(x, ctx, cache, residual, write, out_dtype)
-        if out_dtype is not None and residual is None:
-            return self.forward(x, ctx, cache, None, write).to(out_dtype)
         qkv = project(self.rt, x, self.w_qkv)
         fused = self.position is None or hasattr(self.position, "tables")
         cos = sin = None
@@ -229,7 +227,7 @@ class Attention(Mixer):
                 ctx, write=write, **unit,
             )
             if out is not None:
-                return project(self.rt, out, self.w_out, residual=residual)
+                return project(self.rt, out, self.w_out, out_dtype=out_dtype, residual=residual)
         store = write and fused
         q = ops.qk_norm_rope_store(
             qkv, s.num_heads, s.num_kv_heads, s.head_dim,
@@ -250,7 +248,7 @@ class Attention(Mixer):
             q, cache.k, cache.v, ctx.block_table(cache.group), ctx.seq_of_token, ctx.positions,
             self.scale, s.window, cache.page_size, ctx,
         )
-        return project(self.rt, out, self.w_out, residual=residual)
+        return project(self.rt, out, self.w_out, out_dtype=out_dtype, residual=residual)
 
 
 register_mixer("attention", Attention)
