@@ -73,7 +73,7 @@ def rotate(y, rot, first_position=0):
 
 
 def visible(i, j, window):
-    """Whether position i sees position j: itself and the window - 1 before it."""
+    """Whether position i sees position j."""
     return 0 <= i - j < window
 
 
