@@ -93,6 +93,7 @@ class _Group:
     max_blocks: int = 0  # columns of this group's block table: the pages a request of full context holds
     blocks: Dict[Hashable, List[int]] = field(default_factory=dict)  # request -> page per block, -1 once released
     keep_first: int = 0  # tokens at a request's start that stay readable behind the window: their pages are kept
+    pool: int = 0  # tokens of a block that is not complete yet stay readable behind the window: their pages are kept
 
 
 @dataclass
@@ -165,7 +166,8 @@ class CacheManager:
                     self._group_of[spec.paging()] = gid
                     self.groups.append(_Group(spec.window, PageAllocator(pool_tokens // size), page_size=size,
                                               max_blocks=-(-context // size),
-                                              keep_first=spec.keep_first if spec.window else 0))
+                                              keep_first=spec.keep_first if spec.window else 0,
+                                              pool=spec.pool if spec.window else 0))
                 pools = {name: None for name in spec.pools(size)}
                 if storage:
                     pages = self.groups[gid].allocator.num_pages
@@ -283,6 +285,8 @@ class CacheManager:
                 continue
             # the next query sits at position `length` and sees keys >= length - window + 1
             first_needed = req.length - group.window + 1
+            if group.pool:  # the block that the next token belongs to is still to be summed up
+                first_needed = min(first_needed, req.length // group.pool * group.pool)
             blocks = group.blocks[request]
             kept = -(-group.keep_first // group.page_size)  # blocks that hold tokens every later query still sees
             for b in range(kept, min(len(blocks), max(0, first_needed) // group.page_size)):

@@ -91,7 +91,9 @@ class AttentionSpec:
     # Options that LFM2 leaves at their defaults. Any of them sends the layer to the general attention kernels.
     v_head_dim: Optional[int] = None  # size of a value head; None: head_dim
     softcap: Optional[float] = None  # score <- cap * tanh(score / cap), after the scale
-    distance_bias: bool = False  # score <- score - r1_h * ln(1 + r2_h * (i - j)); r1, r2 are two tensors [heads]
+    # True: score <- score - r1_h * ln(1 + r2_h * (i - j)), r1 and r2 two tensors [heads]; "linear": score <- score -
+    # 2^(-8 (h + 1) / heads) * (i - j) for head h = 0, 1, ..., no tensors
+    distance_bias: Any = False
     keep_first: int = 0  # with a window: the first keep_first positions of a request stay visible behind it
     # one more term in the softmax's denominator, without a key or a value: True: exp(0); "learned": exp(sink_h) with
     # a tensor [heads] of logits, which the scale does not touch
@@ -109,6 +111,14 @@ class AttentionSpec:
     # A number: after the position encoding every head of q and k is divided by sqrt(mean(x^2) + this number) over the
     # whole head, without a weight (where ``qk_norm`` is a norm with a weight in front of the position encoding). None: not.
     qk_unit_eps: Optional[float] = None
+    out_bias: bool = False  # the output product has a bias (``<name>.b`` beside its matrix)
+    # (coef, every): the queries of position p times 1 + coef * ln(floor((p + 1) / every) + 1), after norm and rotation
+    q_temperature: Optional[Tuple[float, int]] = None
+    # With a window: the tokens in front of it are seen as whole blocks of ``pool`` tokens. Block b holds the positions
+    # b * pool .. (b + 1) * pool - 1; position i sees it iff its last position is at most i - window, as one key (the mean
+    # of its tokens' keys as the cache holds them) and one value (the mean of theirs), in the same softmax. Tokens of a
+    # block that is not yet wholly in front of the window, but which the window has passed, are not seen.
+    pool: Optional[int] = None
 
     @property
     def value_dim(self) -> int:
@@ -119,7 +129,7 @@ class AttentionSpec:
         """Whether the layer needs what only the general attention kernels compute."""
         return bool(self.v_head_dim not in (None, self.head_dim) or self.softcap or self.distance_bias or self.keep_first
                     or self.sink or self.gate or self.values_are_keys or getattr(self.position, "interleaved", False)
-                    or self.bias or not self.own_kv
+                    or self.bias or not self.own_kv or self.pool or self.q_temperature
                     or (self.qk_unit_eps is not None and self.head_dim not in (16, 32, 64, 128)))  # sizes of the tensor-core kernels
 
 
@@ -245,6 +255,23 @@ class DecayedLinearAttentionSpec:
 
 
 @dataclass(frozen=True)
+class HGRN2Spec:
+    """Linear attention whose forget gate also decides what is written: S <- diag(f) S + (1 - f) v^T, o = S^T q, per head.
+
+    q = silu(W_q x) [heads x key_dim], v = W_v x [heads x value_dim]; f = l + (1 - l) sigmoid(W_f x + b) per head and key
+    channel, with the lower bound l a tensor [heads * key_dim]. Each head's o is RMS-normed over ``value_dim`` (plain
+    weight shared by the heads) before the output product. The state is float32 and starts at zero."""
+
+    hidden_size: int
+    num_heads: int
+    key_dim: int
+    value_dim: int
+    norm_eps: float
+    kind: str = "hgrn2"
+    names: Mapping[str, str] = field(default_factory=dict)
+
+
+@dataclass(frozen=True)
 class ParallelMixerSpec:
     """Several mixers side by side that read the same input; the result is the sum of ``scale_i * mixer_i(x)``.
 
@@ -273,7 +300,8 @@ class RoutedExpertsSpec:
     (tensors ``shared.{gate,up,down}``) that every token passes, added to the sum, and with ``shared_gate`` times
     sigmoid(W_sg x), one number per token (``shared.sg`` [1, hidden]); ``gated`` False: the experts and the
     shared one have no gate matrix (tensors ``up`` and ``down`` alone) and compute W_down act(W_up x) with ``activation``
-    one of "relu2" (the square of max(z, 0)), "gelu_tanh", "silu"."""
+    one of "relu2" (the square of max(z, 0)), "gelu_tanh", "silu"; ``group_best`` B: a group's score is the sum of its B
+    largest choice scores; ``weight_scale``: every weight times this constant, after the renormalization if there is one."""
 
     hidden_size: int
     intermediate_size: int
@@ -290,6 +318,8 @@ class RoutedExpertsSpec:
     shared_gate: bool = False
     gated: bool = True
     activation: str = "silu"
+    group_best: int = 1
+    weight_scale: float = 1.0
     kind: str = "routed_experts"
     names: Mapping[str, str] = field(default_factory=dict)
 
@@ -351,6 +381,7 @@ class LayerSpec:
     ffn_post_norm: Any = None
     mixer_post_norm_name: Optional[str] = None
     ffn_post_norm_name: Optional[str] = None
+    # "pre_norm" with a multiplier m: h += m * mixer(mixer_norm(h)); h += m * ffn(ffn_norm(h)).
     # What the "parallel" arrangement adds: h += residual_multiplier * (mixer_scale * mixer(n) + ffn_scale * ffn(n))
     # with ONE norm n = mixer_norm(h) that both sublayers read, or, where ``ffn_norm`` is given, a norm for each, both of
     # the same h; the two scales are tensors [hidden] (None: ones).
@@ -369,13 +400,28 @@ class ScheduleEntry:
     is told ``write=False``). Naming a layer in two entries runs its weights twice,
     each time with the cache of its own entry. ``add_embedding``: before the layer runs, the embedding's output (the
     stream as it was in front of the first entry) is added to the stream once more. ``join`` names a tensor
-    W [hidden, 2 hidden]: before the layer runs, the stream x becomes W [x; embedding's output].
+    W [hidden, 2 hidden]: before the layer runs, the stream x becomes W [x; embedding's output]. ``average`` names a
+    tensor w [e + 2] for entry number e: with X_0 the embedding's output and X_(j + 1) the stream as entry j's layer left
+    it (before any averaging behind it), what goes on is sum_j w_j X_j over j = 0 .. e + 1.
     """
 
     layer: int
     cache: Optional[int] = None
     add_embedding: bool = False
     join: Optional[str] = None
+    average: Optional[str] = None
+
+
+@dataclass(frozen=True)
+class BigramSpec:
+    """A second embedding of every token, by the token in front of it: row (previous * mul_prev + token * mul_cur) mod
+    buckets of a table [buckets + 1, hidden] named ``name``; a sequence's first token takes row ``buckets``. The previous
+    token is part of a request's state."""
+
+    name: str
+    buckets: int
+    mul_prev: int
+    mul_cur: int
 
 
 @dataclass(frozen=True)
@@ -401,6 +447,7 @@ class ModelSpec:
     position_table_name: Optional[str] = None
     embedding_norm: Any = None
     embedding_norm_name: Optional[str] = None
+    bigram: Optional[BigramSpec] = None  # added to the embedding's row (before the multiplier)
 
     def run_order(self) -> Tuple[ScheduleEntry, ...]:
         if self.schedule:

@@ -1,13 +1,18 @@
 // Paged softmax attention with options that the specialised kernels do not take: value heads of another size than
-// the keys', a capped score, a logarithmic distance penalty, first tokens that stay visible behind a sliding window,
-// a sink in the softmax's denominator, and a sigmoid gate per head on the output. Prompt portions and decoded tokens
+// the keys', a capped score, a logarithmic or linear distance penalty, first tokens that stay visible behind a sliding
+// window, whole blocks of tokens seen as one key and value in front of it, a sink in the softmax's denominator, and a sigmoid gate per head on the output. Prompt portions and decoded tokens
 // run through the same kernel: one block per (token, key/value head) that serves the group's query heads.
 //
 // Token i of a request sees key j iff j <= i and (window == 0 or i - j < window or j < keep_first). For head h:
 //   s_j = (q . k_j) * scale;  s_j <- cap * tanh(s_j / cap) if cap > 0;  s_j <- s_j - r1_h * ln(1 + r2_h * (i - j)) if r1;
+//   (with r1 alone, no r2: s_j <- s_j - r1_h * (i - j));
 //   p_j = exp(s_j) / (sink + sum_j' exp(s_j'));  out = out_scale * sigmoid(gate_h) * sum_j p_j v_j.
 // The sink is exp(0), or exp(sinks[h]) where a learned logit per head is given. The output's rows have a pitch of
 // their own (ldo elements), so a layer may write its heads into a part of a wider row.
+// With blocks of P tokens (a window, nothing kept, no penalty): besides the window, token i sees every block b with
+// (b + 1) P - 1 <= i - window as one key and one value, the means that pool_blocks made, in the same softmax. Blocks have
+// pages and a block table of their own: a block lies in the page of its last token, in the order of the blocks that end
+// in that page.
 // Scores, weights and sums are float32. The visible keys are walked in tiles of kTile keys whose borders are
 // multiples of kTile counted from position 0 (the kept first tokens come first), so what a token computes, and in
 // which order, depends on its position only: not on how the prompt was cut or on what else is in the batch.
@@ -20,6 +25,11 @@ namespace {
 constexpr int kTile = 128;    // keys per tile = threads per block
 constexpr int kMaxGroup = 16;  // query heads of a key/value head that one block serves at a time
 
+// The factor on the queries of a position: 1 + coef ln(floor((pos + 1) / every) + 1); every 0: none.
+__device__ __forceinline__ float temperature_of(int pos, float coef, int every) {
+  return every > 0 ? fmaf(coef, logf((float)((pos + 1) / every) + 1.f), 1.f) : 1.f;
+}
+
 // One block per token: RMSNorm of every head of q and k over D with a plain weight (or none), then (where tables are
 // given) the rotation of the first `rot` channels of each head by the token's angles, channel 2i with 2i + 1
 // (interleaved) or i with i + rot / 2; q to q_out [N, H * D], k and the untouched v into the pages at the token's
@@ -27,7 +37,7 @@ constexpr int kMaxGroup = 16;  // query heads of a key/value head that one block
 // Where biases are given (float32, one per channel of q, k, v), they are added first, in float32; q, k and v may then
 // be the float32 result of a product (TI) while the pages hold T, so product plus bias is rounded once.
 // unit: there is no norm in front of the rotation; behind it every head of q and k is divided by
-// sqrt(mean of its D squares + eps), without a weight.
+// sqrt(mean of its D squares + eps), without a weight. temp_every > 0: last of all, q times its position's temperature.
 template <typename TI, typename T>
 __global__ void qk_norm_store_kernel(const TI* __restrict__ q, long long ldq, const TI* __restrict__ k, long long ldk,
                                      const TI* __restrict__ v, long long ldv, const float* __restrict__ qw,
@@ -37,7 +47,7 @@ __global__ void qk_norm_store_kernel(const TI* __restrict__ q, long long ldq, co
                                      const int* __restrict__ positions, int page_size, int H, int G, int D, int V, int write,
                                      const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot,
                                      int interleaved, const float* __restrict__ qb, const float* __restrict__ kb,
-                                     const float* __restrict__ vb, int unit) {
+                                     const float* __restrict__ vb, int unit, float temp_coef, int temp_every) {
   const int n = blockIdx.x;
   const int req = seq_of_token[n];
   if (req < 0) return;
@@ -45,6 +55,7 @@ __global__ void qk_norm_store_kernel(const TI* __restrict__ q, long long ldq, co
   const int pos = positions[n];
   const int page = block_table[(size_t)req * max_blocks + pos / page_size];
   const int off = pos % page_size;
+  const float temp = temperature_of(pos, temp_coef, temp_every);
   for (int head = warp; head < H + G; head += warps) {
     const bool is_q = head < H;
     if (!is_q && !write) continue;
@@ -71,10 +82,11 @@ __global__ void qk_norm_store_kernel(const TI* __restrict__ q, long long ldq, co
       ss = warp_sum(ss);
       inv = 1.f / sqrtf(ss / (float)D + eps);
     }
+    const float last = is_q ? temp : 1.f;
     T* dst = is_q ? q_out + ((size_t)n * H + head) * D
                   : k_pool + (((size_t)page * G + (head - H)) * page_size + off) * D;
     if (cos_t == nullptr) {
-      for (int d = lane; d < D; d += 32) dst[d] = from_f32<T>(w != nullptr ? at(d) * inv * w[d] : unit ? at(d) * inv : at(d));
+      for (int d = lane; d < D; d += 32) dst[d] = from_f32<T>((w != nullptr ? at(d) * inv * w[d] : unit ? at(d) * inv : at(d)) * last);
       continue;
     }
     const int half = rot / 2;
@@ -84,10 +96,10 @@ __global__ void qk_norm_store_kernel(const TI* __restrict__ q, long long ldq, co
       if (w != nullptr) { u *= inv * w[a]; x *= inv * w[b]; }
       const float c = cos_t[(size_t)n * half + i], sn = sin_t[(size_t)n * half + i];
       const float ru = fmaf(u, c, -x * sn), rx = fmaf(x, c, u * sn);
-      dst[a] = from_f32<T>(unit ? ru * inv : ru);
-      dst[b] = from_f32<T>(unit ? rx * inv : rx);
+      dst[a] = from_f32<T>((unit ? ru * inv : ru) * last);
+      dst[b] = from_f32<T>((unit ? rx * inv : rx) * last);
     }
-    for (int d = rot + lane; d < D; d += 32) dst[d] = from_f32<T>(w != nullptr ? at(d) * inv * w[d] : unit ? at(d) * inv : at(d));
+    for (int d = rot + lane; d < D; d += 32) dst[d] = from_f32<T>((w != nullptr ? at(d) * inv * w[d] : unit ? at(d) * inv : at(d)) * last);
   }
   if (write) {
     for (int i = threadIdx.x; i < G * V; i += blockDim.x) {
@@ -109,7 +121,8 @@ qk_norm_store8_kernel(const TI* __restrict__ q, long long ldq, const TI* __restr
                       T* __restrict__ k_pool, T* __restrict__ v_pool, const int* __restrict__ block_table, int max_blocks,
                       const int* __restrict__ seq_of_token, const int* __restrict__ positions, int page_size, int H, int G, int D,
                       int V, int write, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot,
-                      const float* __restrict__ qb, const float* __restrict__ kb, const float* __restrict__ vb, int unit, int lph) {
+                      const float* __restrict__ qb, const float* __restrict__ kb, const float* __restrict__ vb, int unit, int lph,
+                      float temp_coef, int temp_every) {
   const int n = blockIdx.x;
   const int req = seq_of_token[n];
   if (req < 0) return;
@@ -174,6 +187,11 @@ qk_norm_store8_kernel(const TI* __restrict__ q, long long ldq, const TI* __restr
 #pragma unroll
     for (int i = 0; i < 8; ++i) x[i] *= inv;
   }
+  if (turns && is_q && temp_every > 0) {
+    const float temp = temperature_of(positions[n], temp_coef, temp_every);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] *= temp;
+  }
   if (turns) {
     if (is_q) store8(q_out + ((size_t)n * H + head) * D + e0, x);
     else store8(k_pool + (row + (long long)g * page_size) * D + e0, x);
@@ -193,6 +211,51 @@ qk_norm_store8_kernel(const TI* __restrict__ q, long long ldq, const TI* __restr
     store8(v_pool + (row + (long long)vg * page_size) * V + j, y);
   }
 }
+
+// One block per token of the step; those of a token that is the last of its block of `block` tokens make the block's key
+// and value per head, the means of its tokens' rows as the pages hold them (float32 sums in the order of the positions),
+// in the block's entry of its own pages. A block that began in earlier steps is read from where they left it.
+template <typename T>
+__global__ void __launch_bounds__(128)
+pool_blocks_kernel(const T* __restrict__ k_pool, const T* __restrict__ v_pool, T* __restrict__ k_blocks, T* __restrict__ v_blocks,
+                   const int* __restrict__ token_table, int token_width, const int* __restrict__ block_table, int block_width,
+                   const int* __restrict__ seq_of_token, const int* __restrict__ positions, int page_size, int block_page,
+                   int entries, int block, int G, int D, int V) {
+  const int n = blockIdx.x;
+  const int req = seq_of_token[n];
+  if (req < 0) return;
+  const int pos = positions[n];
+  if ((pos + 1) % block) return;
+  const int* table = token_table + (size_t)req * token_width;
+  const int page = block_table[(size_t)req * block_width + pos / block_page];
+  const int entry = pos / block - (pos / block_page * block_page) / block;
+  const float inv = 1.f / (float)block;
+  const int first = pos - block + 1, per = D + V;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < G * per; i += gridDim.y * blockDim.x) {
+    const int g = i / per, e = i % per;
+    const T* src = e < D ? k_pool + e : v_pool + (e - D);
+    const int size = e < D ? D : V;
+    float sum = 0.f;
+#pragma unroll 8
+    for (int t = first; t <= pos; ++t) {
+      const long long row = ((long long)table[t / page_size] * G + g) * page_size + t % page_size;
+      sum += to_f32(src[row * size]);
+    }
+    const long long row = ((long long)page * G + g) * entries + entry;
+    if (e < D) k_blocks[row * D + e] = from_f32<T>(sum * inv);
+    else v_blocks[row * V + (e - D)] = from_f32<T>(sum * inv);
+  }
+}
+
+// The blocks that a layer sees in front of its window (block 0: none): their pages, the block table with its width, the
+// tokens and the entries of a page, and the tokens of a block.
+template <typename T>
+struct Blocks {
+  const T* k;
+  const T* v;
+  const int* table;
+  int width, page, entries, block;
+};
 
 // Scores of one key row against `heads` query rows in shared memory: the row is read once, 16 bytes at a time where
 // its size allows, and every head's sum is one ascending chain of fused multiply-adds.
@@ -234,7 +297,8 @@ attention_general_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, 
                          const int* __restrict__ positions, T* __restrict__ out, float scale, int window, int keep_first,
                          float cap, const float* __restrict__ r1, const float* __restrict__ r2, int sink,
                          const TG* __restrict__ gate, long long ldg, int page_size, int H, int G, int D, int V, int row_words,
-                         const float* __restrict__ sinks, float out_scale, long long ldo, long long vpitch, int gate_channels) {
+                         const float* __restrict__ sinks, float out_scale, long long ldo, long long vpitch, int gate_channels,
+                         Blocks<T> blocks) {
   extern __shared__ __align__(16) float smem[];
   const int n = blockIdx.x, g = blockIdx.y;
   const int req = seq_of_token[n];
@@ -269,20 +333,30 @@ attention_general_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, 
     for (int i = tid; i < heads * Vp; i += kTile) acc[i] = 0.f;
     __syncthreads();
 
-    // the two runs of visible keys: [0, kept) and [lo, pos]; tiles start at multiples of kTile
-    for (int run = 0; run < 2; ++run) {
-      const int first = run == 0 ? 0 : lo, last = run == 0 ? kept : pos + 1;  // [first, last)
+    // the runs of visible keys: [0, kept), [lo, pos] and the blocks in front of the window; tiles start at multiples of kTile
+    const int runs = blocks.block > 0 ? 3 : 2;
+    for (int run = 0; run < runs; ++run) {
+      const bool pooled = run == 2;
+      const int first = run == 1 ? lo : 0, last = run == 0 ? kept : run == 1 ? pos + 1 : lo / blocks.block;  // [first, last)
       if (first >= last) continue;
+      const T* keys = pooled ? blocks.k : k_pool;
+      const T* values = pooled ? blocks.v : v_pool;
+      const long long pitch = pooled ? V : vpitch;
       for (int t0 = first / kTile * kTile; t0 < last; t0 += kTile) {
         const int key = t0 + tid;
         const bool seen = key >= first && key < last;
         float sc[kMaxGroup];
         if (seen) {
-          const int page = table[key / page_size];
-          const long long base = ((long long)page * G + g) * page_size + key % page_size;
+          long long base;
+          if (pooled) {
+            const int at = (key * blocks.block + blocks.block - 1) / blocks.page;  // the page of the block's last token
+            base = ((long long)blocks.table[(size_t)req * blocks.width + at] * G + g) * blocks.entries + key - at * blocks.page / blocks.block;
+          } else {
+            base = ((long long)table[key / page_size] * G + g) * page_size + key % page_size;
+          }
           rowbase[tid] = base;
           const float dist = (float)(pos - key);
-          dot_rows(k_pool + (size_t)base * D, qs, D, heads, sc);
+          dot_rows(keys + (size_t)base * D, qs, D, heads, sc);
 #pragma unroll
           for (int a = 0; a < kMaxGroup; ++a) {
             if (a < heads) {
@@ -290,7 +364,7 @@ attention_general_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, 
               if (cap > 0.f) s = cap * tanhf(s / cap);
               if (r1 != nullptr) {
                 const int h = g * group + h0 + a;
-                s -= r1[h] * log1pf(r2[h] * dist);
+                s -= r2 != nullptr ? r1[h] * log1pf(r2[h] * dist) : r1[h] * dist;
               }
               sc[a] = s;
             }
@@ -337,7 +411,7 @@ attention_general_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, 
           for (int a = 0; a < kMaxGroup; ++a) add[a] = 0.f;
 #pragma unroll 8
           for (int t = begin; t < count; ++t) {  // (the rows' places were found with the scores: these loads do not wait on one another)
-            const float vv = to_f32(v_pool[(size_t)rowbase[t] * vpitch + c]);
+            const float vv = to_f32(values[(size_t)rowbase[t] * pitch + c]);
 #pragma unroll
             for (int a = 0; a < kMaxGroup; ++a)
               if (a < heads) add[a] = fmaf(pw[a * kTile + t], vv, add[a]);
@@ -375,7 +449,7 @@ AKAS_API int akas_qk_norm_store(const void* q, long long ldq, const void* k, lon
                                 const int* block_table, int max_blocks, const int* seq_of_token, const int* positions,
                                 int page_size, int N, int H, int G, int D, int V, int write, int dtype, const float* cos_t,
                                 const float* sin_t, int rot, int interleaved, int in_dtype, const float* qb, const float* kb,
-                                const float* vb, int unit, cudaStream_t stream) {
+                                const float* vb, int unit, float temp_coef, int temp_every, cudaStream_t stream) {
   if (N <= 0) return 0;
   if (unit && (qw != nullptr || kw != nullptr)) return (int)cudaErrorInvalidValue;
   if ((qw == nullptr) != (kw == nullptr)) return (int)cudaErrorInvalidValue;
@@ -391,7 +465,8 @@ AKAS_API int akas_qk_norm_store(const void* q, long long ldq, const void* k, lon
 #define AKAS_STORE8(TI, T)                                                                                                    \
   return launch_ordinary(qk_norm_store8_kernel<TI, T>, grid, dim3(128), 0, stream, (const TI*)q, ldq, (const TI*)k, ldk,      \
                          (const TI*)v, ldv, qw, kw, eps, (T*)q_out, (T*)k_pool, (T*)v_pool, block_table, max_blocks,          \
-                         seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, qb, kb, vb, unit, lph)
+                         seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, qb, kb, vb, unit, lph,     \
+                         temp_coef, temp_every)
     if (dtype == AKAS_F32) AKAS_STORE8(float, float);
     if (in_dtype == AKAS_F32) AKAS_STORE8(float, bf16);
     AKAS_STORE8(bf16, bf16);
@@ -402,14 +477,14 @@ AKAS_API int akas_qk_norm_store(const void* q, long long ldq, const void* k, lon
   if (dtype == AKAS_F32)
     return launch_ordinary(qk_norm_store_kernel<float, float>, dim3(N), dim3(128), 0, stream, (const float*)q, ldq, (const float*)k, ldk,
                           (const float*)v, ldv, qw, kw, eps, (float*)q_out, (float*)k_pool, (float*)v_pool, block_table,
-                          max_blocks, seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb, unit);
+                          max_blocks, seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb, unit, temp_coef, temp_every);
   if (in_dtype == AKAS_F32)
     return launch_ordinary(qk_norm_store_kernel<float, bf16>, dim3(N), dim3(128), 0, stream, (const float*)q, ldq, (const float*)k, ldk,
                           (const float*)v, ldv, qw, kw, eps, (bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool, block_table, max_blocks,
-                          seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb, unit);
+                          seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb, unit, temp_coef, temp_every);
   return launch_ordinary(qk_norm_store_kernel<bf16, bf16>, dim3(N), dim3(128), 0, stream, (const bf16*)q, ldq, (const bf16*)k, ldk,
                         (const bf16*)v, ldv, qw, kw, eps, (bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool, block_table, max_blocks,
-                        seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb, unit);
+                        seq_of_token, positions, page_size, H, G, D, V, write, cos_t, sin_t, rot, interleaved, qb, kb, vb, unit, temp_coef, temp_every);
 }
 
 template <typename T, typename TG>
@@ -417,7 +492,8 @@ static int launch_general(const void* q, const void* k_pool, const void* v_pool,
                           const int* seq_of_token, const int* positions, void* out, float scale, int window, int keep_first,
                           float cap, const float* r1, const float* r2, int sink, const void* gate, long long ldg,
                           int page_size, int N, int H, int G, int D, int V, const float* sinks, float out_scale,
-                          long long ldo, long long vpitch, int gate_channels, cudaStream_t stream) {
+                          long long ldo, long long vpitch, int gate_channels, const void* k_blocks, const void* v_blocks,
+                          const int* blocks_table, int blocks_width, int block_page, int block, cudaStream_t stream) {
   const int Vp = (V + kTile - 1) / kTile * kTile;
   const int row_words = (kMaxGroup * D + kMaxGroup * kTile + kMaxGroup * 4 + kMaxGroup * 2 + kMaxGroup * Vp + 1) / 2 * 2;
   const size_t smem = sizeof(float) * (size_t)row_words + sizeof(long long) * kTile;
@@ -432,7 +508,9 @@ static int launch_general(const void* q, const void* k_pool, const void* v_pool,
   }
   return launch_ordinary(attention_general_kernel<T, TG>, dim3(N, G), dim3(kTile), smem, stream, (const T*)q, (const T*)k_pool,
                         (const T*)v_pool, block_table, max_blocks, seq_of_token, positions, (T*)out, scale, window, keep_first,
-                        cap, r1, r2, sink, (const TG*)gate, ldg, page_size, H, G, D, V, row_words, sinks, out_scale, ldo, vpitch, gate_channels);
+                        cap, r1, r2, sink, (const TG*)gate, ldg, page_size, H, G, D, V, row_words, sinks, out_scale, ldo, vpitch, gate_channels,
+                        Blocks<T>{(const T*)k_blocks, (const T*)v_blocks, blocks_table, blocks_width, block_page,
+                                  block > 0 ? (block_page + block - 1) / block : 0, block});
 }
 
 AKAS_API int akas_attention_general(const void* q, const void* k_pool, const void* v_pool, const int* block_table,
@@ -440,16 +518,43 @@ AKAS_API int akas_attention_general(const void* q, const void* k_pool, const voi
                                     int window, int keep_first, float cap, const float* r1, const float* r2, int sink,
                                     const void* gate, long long ldg, int page_size, int N, int H, int G, int D, int V,
                                     int dtype, const float* sinks, float out_scale, long long ldo, long long vpitch,
-                                    int gate_channels, int gate_dtype, cudaStream_t stream) {
+                                    int gate_channels, int gate_dtype, const void* k_blocks, const void* v_blocks,
+                                    const int* blocks_table, int blocks_width, int block_page, int block, cudaStream_t stream) {
   if (N <= 0) return 0;
   if (G <= 0 || H % G || vpitch < V) return (int)cudaErrorInvalidValue;
+  // blocks: a window in front of which they lie, and none of the options that the walk over them does not know
+  if (block < 0 || (block > 0 && (window <= 0 || keep_first > 0 || r1 != nullptr || block_page <= 0 || k_blocks == nullptr ||
+                                  v_blocks == nullptr || blocks_table == nullptr)))
+    return (int)cudaErrorInvalidValue;
   if (dtype == AKAS_BF16 && gate != nullptr && gate_dtype == AKAS_F32)  // the gate's logits as a float32 product left them
     return launch_general<bf16, float>(q, k_pool, v_pool, block_table, max_blocks, seq_of_token, positions, out, scale, window,
-                                       keep_first, cap, r1, r2, sink, gate, ldg, page_size, N, H, G, D, V, sinks, out_scale, ldo, vpitch, gate_channels, stream);
+                                       keep_first, cap, r1, r2, sink, gate, ldg, page_size, N, H, G, D, V, sinks, out_scale, ldo, vpitch, gate_channels, k_blocks, v_blocks,
+                                        blocks_table, blocks_width, block_page, block, stream);
   if (dtype == AKAS_F32 && gate != nullptr && gate_dtype != AKAS_F32) return (int)cudaErrorInvalidValue;
   if (dtype == AKAS_F32)
     return launch_general<float, float>(q, k_pool, v_pool, block_table, max_blocks, seq_of_token, positions, out, scale, window,
-                                        keep_first, cap, r1, r2, sink, gate, ldg, page_size, N, H, G, D, V, sinks, out_scale, ldo, vpitch, gate_channels, stream);
+                                        keep_first, cap, r1, r2, sink, gate, ldg, page_size, N, H, G, D, V, sinks, out_scale, ldo, vpitch, gate_channels, k_blocks, v_blocks,
+                                        blocks_table, blocks_width, block_page, block, stream);
   return launch_general<bf16, bf16>(q, k_pool, v_pool, block_table, max_blocks, seq_of_token, positions, out, scale, window,
-                                    keep_first, cap, r1, r2, sink, gate, ldg, page_size, N, H, G, D, V, sinks, out_scale, ldo, vpitch, gate_channels, stream);
+                                    keep_first, cap, r1, r2, sink, gate, ldg, page_size, N, H, G, D, V, sinks, out_scale, ldo, vpitch, gate_channels, k_blocks, v_blocks,
+                                        blocks_table, blocks_width, block_page, block, stream);
+}
+
+// The means of every block of `block` tokens that a token of this step completes; block_page: tokens of a page of the
+// blocks' pools, whose pages hold ceil(block_page / block) entries.
+AKAS_API int akas_pool_blocks(const void* k_pool, const void* v_pool, void* k_blocks, void* v_blocks, const int* token_table,
+                              int token_width, const int* block_table, int block_width, const int* seq_of_token,
+                              const int* positions, int page_size, int block_page, int block, int N, int G, int D, int V, int dtype,
+                              cudaStream_t stream) {
+  if (N <= 0) return 0;
+  if (block <= 0 || block_page <= 0 || page_size <= 0) return (int)cudaErrorInvalidValue;
+  const int entries = (block_page + block - 1) / block;
+  const dim3 grid(N, N <= 64 ? max(1, min(16, (G * (D + V) + 127) / 128)) : 1);
+  if (dtype == AKAS_F32)
+    return launch_ordinary(pool_blocks_kernel<float>, grid, dim3(128), 0, stream, (const float*)k_pool, (const float*)v_pool,
+                           (float*)k_blocks, (float*)v_blocks, token_table, token_width, block_table, block_width, seq_of_token,
+                           positions, page_size, block_page, entries, block, G, D, V);
+  return launch_ordinary(pool_blocks_kernel<bf16>, grid, dim3(128), 0, stream, (const bf16*)k_pool, (const bf16*)v_pool,
+                         (bf16*)k_blocks, (bf16*)v_blocks, token_table, token_width, block_table, block_width, seq_of_token,
+                         positions, page_size, block_page, entries, block, G, D, V);
 }

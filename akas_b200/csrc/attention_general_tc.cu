@@ -2,11 +2,12 @@
 // tensor cores, flash-attention style: the walk of attention_prefill.cu with the options as arguments.
 //
 // One block per (tile of 64 consecutive query tokens of one request, query head); 4 warps of 16 query rows. The block
-// walks 64-key tiles aligned to absolute position 0: first the tiles of the kept first tokens that lie before its
+// walks 64-key tiles aligned to absolute position 0: first the tiles of the blocks of tokens in front of its window (where
+// the layer sees such blocks, 64 blocks a tile), then those of the kept first tokens that lie before its
 // window, then from the first key its window reaches to its last query's own position. K rows [DK] and V rows [DV]
 // come from the pages by 16-byte cp.async copies, two tiles in flight; columns beyond the real head sizes (which need
 // only be multiples of 8) are zero in shared memory. S = Q.K^T and O += P.V are mma.sync m16n8k16; between them, in
-// float32 registers: scale, cap * tanh(s / cap), minus r1 * ln(1 + r2 * distance), the mask by absolute positions,
+// float32 registers: scale, cap * tanh(s / cap), minus r1 * ln(1 + r2 * distance) or r1 * distance, the mask by absolute positions,
 // and the running maximum and sum, which start at the sink's logit (0, or a learned number per head) and 1 where the
 // softmax has a sink. The head's output is multiplied by sigmoid(gate) and by a constant on its way out, into rows
 // whose pitch is the caller's.
@@ -55,6 +56,12 @@ struct Options {
   long long vpitch;    // elements between two value rows in the pages (V, or more where a row holds more than the value)
   int gate_channels;   // the gate has one logit per output channel [H * V] of a token, not one per head [H]
   int gate_f32;        // the gate's logits are float32 (the rows of a product that left float32)
+  // blocks of `block` tokens seen as one key and value in front of the window (0: none): pages of `entries` blocks for
+  // `bpage` tokens, a block in the page of its last token; a block table of their own, `bwidth` pages a request
+  const bf16* k_blocks;
+  const bf16* v_blocks;
+  const int* btable;
+  int bwidth, bpage, entries, block;
 };
 
 __device__ __forceinline__ float gate_at(const Options& opt, size_t at) {  // sigmoid of the logit at an element offset
@@ -124,18 +131,46 @@ general_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_po
   const int first_key = window > 0 ? max(0, pos0 - window + 1) : 0;
   const int kt0 = first_key / BK, kt1 = last_key / BK;
   const int kept_tiles = min((keep + BK - 1) / BK, kt0);  // tiles of kept tokens that lie wholly before the window's first
-  const int total = kept_tiles + (kt1 - kt0 + 1);
+  // blocks that the block's last query sees, and their tiles (numbered -1, -2, ... below)
+  auto blocks_seen = [&](int p) { return opt.block > 0 ? max(0, p - window + 1) / opt.block : 0; };
+  const int last_blocks = blocks_seen(last_key);
+  const int block_tiles = (last_blocks + BK - 1) / BK;
+  const int total = block_tiles + kept_tiles + (kt1 - kt0 + 1);
   int i_begin = 0, i_end = total;  // the tiles this block walks: all, or its part of them
   if (splits > 1) {
     const int per = (total + splits - 1) / splits;
     i_begin = min(total, (int)blockIdx.z * per);
     i_end = min(total, i_begin + per);
   }
-  auto tile_of = [&](int i) { return i < kept_tiles ? i : kt0 + (i - kept_tiles); };
+  auto tile_of = [&](int i) {
+    if (i < block_tiles) return -1 - i;
+    i -= block_tiles;
+    return i < kept_tiles ? i : kt0 + (i - kept_tiles);
+  };
 
   auto load_tile = [&](int kt, int stage) {
     bf16* ks_ = k_s + stage * BK * KSTRIDE;
     bf16* vs_ = v_s + stage * BK * VSTRIDE;
+    if (kt < 0) {
+      const int b0 = (-1 - kt) * BK;
+      for (int c = tid; c < BK * (KCH + VCH); c += WARPS * 32) {
+        const int row = c / (KCH + VCH), ch = c % (KCH + VCH);
+        const int b = b0 + row;
+        const int at = (b * opt.block + opt.block - 1) / opt.bpage;  // the page of the block's last token
+        int page = -1;
+        if (b < last_blocks) page = opt.btable[(size_t)r * opt.bwidth + at];
+        const size_t base = page >= 0 ? ((size_t)page * KH + kvh) * opt.entries + b - at * opt.bpage / opt.block : 0;
+        if (ch < KCH) {
+          const int col = ch * 8;
+          cp_async16(ks_ + row * KSTRIDE + col, opt.k_blocks + base * D + min(col, D - 8), page >= 0 && col < D ? 16 : 0);
+        } else {
+          const int col = (ch - KCH) * 8;
+          cp_async16(vs_ + row * VSTRIDE + col, opt.v_blocks + base * V + min(col, V - 8), page >= 0 && col < V ? 16 : 0);
+        }
+      }
+      cp_async_commit();
+      return;
+    }
     for (int c = tid; c < BK * (KCH + VCH); c += WARPS * 32) {
       const int row = c / (KCH + VCH), ch = c % (KCH + VCH);
       const int key = kt * BK + row;
@@ -166,10 +201,12 @@ general_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_po
   m_run[0] = !sunk ? -INFINITY : opt.sinks != nullptr ? opt.sinks[head2[0]] * kLog2e : 0.f;
   m_run[1] = !sunk ? -INFINITY : opt.sinks != nullptr ? opt.sinks[head2[1]] * kLog2e : 0.f;
   l_run[0] = l_run[1] = sunk && t == 0 ? 1.f : 0.f;
-  const bool biased = opt.r1 != nullptr;
+  const bool biased = opt.r1 != nullptr, linear = biased && opt.r2 == nullptr;
   // r1 ln(1 + r2 d) in units of log2 e is r1 lg2(1 + r2 d): the two factors ln 2 and log2 e cancel
-  const float r1[2] = {biased ? opt.r1[head2[0]] : 0.f, biased ? opt.r1[head2[1]] : 0.f};
-  const float r2[2] = {biased ? opt.r2[head2[0]] : 0.f, biased ? opt.r2[head2[1]] : 0.f};
+  // (the linear penalty r1 d keeps the factor)
+  const float unit = linear ? kLog2e : 1.f;
+  const float r1[2] = {biased ? unit * opt.r1[head2[0]] : 0.f, biased ? unit * opt.r1[head2[1]] : 0.f};
+  const float r2[2] = {biased && !linear ? opt.r2[head2[0]] : 0.f, biased && !linear ? opt.r2[head2[1]] : 0.f};
   const float inv_cap = opt.cap > 0.f ? 1.f / opt.cap : 0.f;
   const float cap2 = opt.cap * kLog2e, scale2 = opt.scale * kLog2e;
 
@@ -215,17 +252,24 @@ general_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_po
     float m_new[2] = {m_run[0], m_run[1]};
     // A tile without kept first tokens (all but a request's first few): a key is seen iff 0 <= distance < window, and
     // the penalty of every distance in it is in the table (where there is a penalty, there must be a table).
-    const bool fast = kt * BK >= keep && (!biased || table > 0);
+    // A tile of blocks: a block is seen iff its number is below the count of blocks in front of the query's window; what
+    // takes the distance's place is how far below.
+    const bool pooled = kt < 0;
+    const bool fast = pooled || (kt * BK >= keep && (!biased || linear || table > 0));
     if (fast) {
-      const int dbase[2] = {qpos[0] - (kt * BK + 2 * t), qpos[1] - (kt * BK + 2 * t)};
+      const int origin = (pooled ? -1 - kt : kt) * BK + 2 * t;
+      const int dbase[2] = {(pooled ? blocks_seen(qpos[0]) - 1 : qpos[0]) - origin, (pooled ? blocks_seen(qpos[1]) - 1 : qpos[1]) - origin};
+      const unsigned limit = pooled ? 0x7fffffffu : (unsigned)wlimit;
+      const float fbase[2] = {(float)dbase[0], (float)dbase[1]};
 #pragma unroll
       for (int nb = 0; nb < BK / 8; ++nb) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int dist = dbase[e >> 1] - (nb * 8 + (e & 1));
           float x = opt.cap > 0.f ? cap2 * fast_tanh(s[nb][e] * scale_cap) : s[nb][e] * scale2;
-          if (biased) x -= penalty[dist];
-          s[nb][e] = (unsigned)dist < (unsigned)wlimit ? x : -INFINITY;
+          if (linear) x = fmaf(-r1[e >> 1], fbase[e >> 1] - (float)(nb * 8 + (e & 1)), x);
+          else if (biased) x -= penalty[dist];
+          s[nb][e] = (unsigned)dist < limit ? x : -INFINITY;
           m_new[e >> 1] = fmaxf(m_new[e >> 1], s[nb][e]);
         }
       }
@@ -238,7 +282,8 @@ general_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_po
           const int qp = qpos[e >> 1];
           const bool seen = key <= qp && (window <= 0 || key > qp - window || key < keep);
           float x = opt.cap > 0.f ? cap2 * fast_tanh(s[nb][e] * scale_cap) : s[nb][e] * scale2;
-          if (biased) x -= r1[e >> 1] * fast_log2(fmaf(r2[e >> 1], (float)max(qp - key, 0), 1.f));
+          if (linear) x -= r1[e >> 1] * (float)max(qp - key, 0);
+          else if (biased) x -= r1[e >> 1] * fast_log2(fmaf(r2[e >> 1], (float)max(qp - key, 0), 1.f));
           s[nb][e] = seen ? x : -INFINITY;
           m_new[e >> 1] = fmaxf(m_new[e >> 1], s[nb][e]);
         }
@@ -388,7 +433,7 @@ int launch(const void* q, const void* k_pool, const void* v_pool, const int* blo
            int KH, int D, int V, int R, int packed, float* partial, int splits, cudaStream_t stream) {
   // the table of distance penalties: for unpacked launches (one head a block) with a window of at most kTableMost keys
   constexpr int kTableMost = 8192;
-  const int table = !packed && opt.r1 != nullptr && opt.window > 0 && opt.window <= kTableMost ? opt.window : 0;
+  const int table = !packed && opt.r1 != nullptr && opt.r2 != nullptr && opt.window > 0 && opt.window <= kTableMost ? opt.window : 0;
   constexpr int tiles_bytes = 2 * BK * ((DKP + 8) + (DVP + 8)) * (int)sizeof(bf16);
   const int smem = tiles_bytes + (table ? table + kTableBefore + kTableAfter : 0) * (int)sizeof(float);
   static bool configured[64] = {};
@@ -421,7 +466,9 @@ AKAS_API int akas_attention_general_tc(const void* q, const void* k_pool, const 
                                        int window, int keep_first, float cap, const float* r1, const float* r2, int sink,
                                        const void* gate, long long ldg, int page_size, int tiles, int H, int KH, int D, int V,
                                        int R, int packed, const float* sinks, float out_scale, long long ldo, float* partial,
-                                       int splits, long long vpitch, int gate_channels, int gate_dtype, cudaStream_t stream) {
+                                       int splits, long long vpitch, int gate_channels, int gate_dtype, const void* k_blocks,
+                                       const void* v_blocks, const int* blocks_table, int blocks_width, int block_page, int block,
+                                       cudaStream_t stream) {
   if (!akas_attention_general_tc_takes(D, V)) return 3999;
   if (ldo % 2 || vpitch % 8 || vpitch < V) return 3999;
   // parts: packed launches only; partial holds (first token of the launch + R) * H * splits * (V + 2) floats
@@ -429,7 +476,13 @@ AKAS_API int akas_attention_general_tc(const void* q, const void* k_pool, const 
   if (packed && (KH <= 0 || H / KH > BQ || tiles != R)) return 3999;
   if (KH <= 0 || H % KH || tiles > 65535 || R <= 0) return (int)cudaErrorInvalidValue;
   if (tiles <= 0) return 0;
-  const Options opt = {scale, cap, r1, r2, window, keep_first, sink, gate, ldg, sinks, out_scale, ldo, vpitch, gate_channels, gate_dtype == AKAS_F32};
+  if (block < 0 || (block > 0 && (window <= 0 || keep_first > 0 || r1 != nullptr || block_page <= 0 || k_blocks == nullptr ||
+                                  v_blocks == nullptr || blocks_table == nullptr)))
+    return (int)cudaErrorInvalidValue;
+  if (((uintptr_t)k_blocks | (uintptr_t)v_blocks) % 16) return 3999;
+  const Options opt = {scale, cap, r1, r2, window, keep_first, sink, gate, ldg, sinks, out_scale, ldo, vpitch, gate_channels, gate_dtype == AKAS_F32,
+                       (const bf16*)k_blocks, (const bf16*)v_blocks, blocks_table, blocks_width, block_page,
+                       block > 0 ? (block_page + block - 1) / block : 0, block};
   const int dk = (D + 31) / 32, dv = (V + 31) / 32;
 #define AKAS_TC(A, B)                                                                                                   \
   if (dk == A && dv == B)                                                                                               \

@@ -1,4 +1,4 @@
-// Embedding gather, RMSNorm (optionally of gathered rows), SwiGLU and the reset of state rows.
+// Embedding gather (alone and with a row per pair of neighbouring tokens), weighted sums over layers' results, RMSNorm (optionally of gathered rows), SwiGLU and the reset of state rows.
 //
 // The residual stream is float32 in both precisions: the embedding writes float32, RMSNorm reads
 // it and writes the compute dtype that the next matrix product takes. All sums are float32.
@@ -25,6 +25,171 @@ AKAS_API int akas_embedding(const int* tokens, const void* table, float* out, in
   if (dtype == AKAS_F32)
     return launch_chained(embedding_kernel<float>, dim3(N), dim3(threads), 0, stream, tokens, (const float*)table, out, C);
   return launch_chained(embedding_kernel<bf16>, dim3(N), dim3(threads), 0, stream, tokens, (const bf16*)table, out, C);
+}
+
+// out[n, :] = float(table[token, :]) + float(pairs[row, :]) with row = (previous * mul_prev + token * mul_cur) mod buckets,
+// previous the token in front of token n in its request; row `buckets` for a request's first token. The last token of
+// the steps before lies in state[slot] plus one (0: none yet); the block of a request's first token of this step, the
+// only one that reads it, leaves the step's last token there. Tokens of no request (seq -1) get their row of `table`
+// alone. copy (or null): the result once more.
+template <typename T>
+__global__ void bigram_embedding_kernel(const int* __restrict__ tokens, const T* __restrict__ table, const T* __restrict__ pairs,
+                                        long long mul_prev, long long mul_cur, int buckets, int* __restrict__ state,
+                                        const int* __restrict__ cu_seqlens, const int* __restrict__ seq_of_token,
+                                        const int* __restrict__ slots, float* __restrict__ out, float* __restrict__ copy, int C) {
+  const int n = blockIdx.x;
+  const int token = tokens[n], req = seq_of_token[n];
+  const T* row = table + (size_t)token * C;
+  const T* pair = nullptr;
+  if (req >= 0) {
+    const int first = cu_seqlens[req];
+    const int slot = slots[req];
+    const int previous = n > first ? tokens[n - 1] : state[slot] - 1;
+    const long long at = previous < 0 ? buckets : ((long long)previous * mul_prev + (long long)token * mul_cur) % buckets;
+    pair = pairs + (size_t)at * C;
+    if (n == first) {
+      __syncthreads();  // every thread has read the state
+      if (threadIdx.x == 0) state[slot] = tokens[cu_seqlens[req + 1] - 1] + 1;
+    }
+  }
+  for (int c = threadIdx.x; c < C; c += blockDim.x) {
+    float v = to_f32(row[c]);
+    if (pair != nullptr) v += to_f32(pair[c]);
+    out[(size_t)n * C + c] = v;
+    if (copy != nullptr) copy[(size_t)n * C + c] = v;
+  }
+}
+
+AKAS_API int akas_bigram_embedding(const int* tokens, const void* table, const void* pairs, long long mul_prev, long long mul_cur,
+                                   int buckets, int* state, const int* cu_seqlens, const int* seq_of_token, const int* slots,
+                                   float* out, float* copy, int N, int C, int dtype, cudaStream_t stream) {
+  if (N <= 0) return 0;
+  if (buckets <= 0) return (int)cudaErrorInvalidValue;
+  const int threads = C >= 1024 ? 256 : 128;
+  if (dtype == AKAS_F32)
+    return launch_ordinary(bigram_embedding_kernel<float>, dim3(N), dim3(threads), 0, stream, tokens, (const float*)table,
+                           (const float*)pairs, mul_prev, mul_cur, buckets, state, cu_seqlens, seq_of_token, slots, out, copy, C);
+  return launch_ordinary(bigram_embedding_kernel<bf16>, dim3(N), dim3(threads), 0, stream, tokens, (const bf16*)table,
+                         (const bf16*)pairs, mul_prev, mul_cur, buckets, state, cu_seqlens, seq_of_token, slots, out, copy, C);
+}
+
+// out[i, :] = sum over j < count of w[j] * history[j][row(i), :], float32, in ascending j; history's layers lie `stride`
+// floats apart; row(i) = rows[i] if rows else i. V channels a thread (4: rows on 16 bytes).
+template <int V>
+__global__ void __launch_bounds__(128)
+depth_average_kernel(const float* __restrict__ history, long long stride, int count, const float* __restrict__ w,
+                     float* __restrict__ out, const int* __restrict__ rows, int C, long long items) {
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= items) return;
+  const int per_row = C / V;
+  const long long m = i / per_row;
+  const int c = (int)(i % per_row) * V;
+  const float* src = history + (rows != nullptr ? (long long)rows[m] : m) * C + c;
+  if (V == 4) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int j = 0; j < count; ++j) {
+      const float4 v = *reinterpret_cast<const float4*>(src + j * stride);
+      const float a = w[j];
+      acc.x = fmaf(a, v.x, acc.x); acc.y = fmaf(a, v.y, acc.y); acc.z = fmaf(a, v.z, acc.z); acc.w = fmaf(a, v.w, acc.w);
+    }
+    *reinterpret_cast<float4*>(out + m * C + c) = acc;
+  } else {
+    float acc = 0.f;
+    for (int j = 0; j < count; ++j) acc = fmaf(w[j], src[j * stride], acc);
+    out[m * C + c] = acc;
+  }
+}
+
+// The same and, in the same pass, y[i, :] = the RMSNorm of that row with weight nw: one block per row, which stays in
+// registers between the sum of squares and the scaling. C a multiple of 4, at most 8192: PER groups of 4 a thread.
+template <typename TO, int PER>
+__global__ void __launch_bounds__(512)
+depth_average_norm_kernel(const float* __restrict__ history, long long stride, int count, const float* __restrict__ w,
+                          float* __restrict__ out, const int* __restrict__ rows, int C, const float* __restrict__ nw, float eps,
+                          int zero_centered, TO* __restrict__ y) {
+  __shared__ float scratch[32];
+  const size_t m = blockIdx.x;
+  const float* src = history + (rows != nullptr ? (size_t)rows[m] : m) * C;
+  float acc[PER][4];
+#pragma unroll
+  for (int p = 0; p < PER; ++p) acc[p][0] = acc[p][1] = acc[p][2] = acc[p][3] = 0.f;
+  // (in chunks of 4 layers whose loads are asked for together)
+  for (int j0 = 0; j0 < count; j0 += 4) {
+    float4 v[PER][4];
+    float a[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      a[e] = j0 + e < count ? w[j0 + e] : 0.f;
+#pragma unroll
+      for (int p = 0; p < PER; ++p) {
+        const int c = (p * blockDim.x + threadIdx.x) * 4;
+        v[p][e] = j0 + e < count && c < C ? *reinterpret_cast<const float4*>(src + (j0 + e) * stride + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+#pragma unroll
+      for (int p = 0; p < PER; ++p) {
+        acc[p][0] = fmaf(a[e], v[p][e].x, acc[p][0]); acc[p][1] = fmaf(a[e], v[p][e].y, acc[p][1]);
+        acc[p][2] = fmaf(a[e], v[p][e].z, acc[p][2]); acc[p][3] = fmaf(a[e], v[p][e].w, acc[p][3]);
+      }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int p = 0; p < PER; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * 4;
+    if (c < C) *reinterpret_cast<float4*>(out + m * C + c) = make_float4(acc[p][0], acc[p][1], acc[p][2], acc[p][3]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) ss = fmaf(acc[p][e], acc[p][e], ss);
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.f / sqrtf(ss / (float)C + eps);
+#pragma unroll
+  for (int p = 0; p < PER; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * 4;
+    if (c < C) {
+      const float4 g = *reinterpret_cast<const float4*>(nw + c);
+      const float shift = zero_centered ? 1.f : 0.f;
+      const float r[4] = {acc[p][0] * inv * (g.x + shift), acc[p][1] * inv * (g.y + shift), acc[p][2] * inv * (g.z + shift),
+                          acc[p][3] * inv * (g.w + shift)};
+      TO* dst = y + m * C + c;
+      if (sizeof(TO) == 4) {
+        *reinterpret_cast<float4*>(dst) = make_float4(r[0], r[1], r[2], r[3]);
+      } else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(r[0], r[1]), hi = __floats2bfloat162_rn(r[2], r[3]);
+        *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+      }
+    }
+  }
+}
+
+AKAS_API int akas_depth_average(const float* history, long long stride, int count, const float* w, float* out, const int* rows,
+                                int M, int C, cudaStream_t stream) {
+  if (M <= 0 || C <= 0) return 0;
+  const bool vec = C % 4 == 0 && stride % 4 == 0 && ((uintptr_t)history | (uintptr_t)out) % 16 == 0;
+  const long long items = (long long)M * (vec ? C / 4 : C);
+  const dim3 grid((unsigned)((items + 127) / 128));
+  return vec ? launch_ordinary(depth_average_kernel<4>, grid, dim3(128), 0, stream, history, stride, count, w, out, rows, C, items)
+             : launch_ordinary(depth_average_kernel<1>, grid, dim3(128), 0, stream, history, stride, count, w, out, rows, C, items);
+}
+
+// 3999: sizes that the fused kernel does not take.
+AKAS_API int akas_depth_average_norm(const float* history, long long stride, int count, const float* w, float* out, const int* rows,
+                                     int M, int C, const float* nw, float eps, int zero_centered, void* y, int out_dtype,
+                                     cudaStream_t stream) {
+  if (C % 4 || C > 8192 || stride % 4 || ((uintptr_t)history | (uintptr_t)out | (uintptr_t)nw | (uintptr_t)y) % 16) return 3999;
+  if (M <= 0) return 0;
+  const int groups = C / 4;
+  const int threads = groups >= 512 ? 512 : (groups + 31) / 32 * 32;
+#define AKAS_AVERAGE(TO, P)                                                                                                        \
+  return launch_ordinary(depth_average_norm_kernel<TO, P>, dim3(M), dim3(threads), 0, stream, history, stride, count, w, out, rows, C, nw, \
+                         eps, zero_centered, (TO*)y)
+  if (out_dtype == AKAS_F32) { if (groups <= 512) AKAS_AVERAGE(float, 1); else if (groups <= 1024) AKAS_AVERAGE(float, 2); else AKAS_AVERAGE(float, 4); }
+  if (groups <= 512) AKAS_AVERAGE(bf16, 1);
+  if (groups <= 1024) AKAS_AVERAGE(bf16, 2);
+  AKAS_AVERAGE(bf16, 4);
+#undef AKAS_AVERAGE
 }
 
 // y[i, :] = x[row(i), :] * rsqrt(mean(x^2) + eps) * (w or 1 + w); row(i) = rows[i] if rows else i.

@@ -8,7 +8,9 @@
 // they have no matrices and return their input. Options: `sigmoid`, s = 1 / (1 + exp(-z)) per output instead of the
 // softmax; no correction (a null pointer); `renorm` 0, the weights are the chosen s as they are; `extra` more rows of
 // W_r behind the R that compete, whose sigmoids are returned beside the choice (gates that read the router's input).
-// Without a correction the choice goes by the logits themselves, which order as the scores do.
+// Without a correction the choice goes by the logits themselves, which order as the scores do. `group_best` B > 1: a
+// group's score is the sum of its B largest choice scores (and the choice then goes by the scores in any case);
+// `wscale`: every weight times this constant.
 //
 // Experts, token by token (moe_gate_up, moe_down): act[pair] = silu(W_gate h) * (W_up h) for every (token, chosen
 // real expert) pair, then out[n] = sum over the token's chosen outputs of weight * (W_down act, or h for an identity
@@ -41,7 +43,7 @@ template <typename T>
 __global__ void __launch_bounds__(kRouteTokens * 32)
 moe_route_kernel(const T* __restrict__ h, long long ldh, const float* __restrict__ w, const float* __restrict__ correction,
                  int* __restrict__ chosen, float* __restrict__ weights, int N, int C, int RC, int groups, int keep, int top,
-                 int sigmoid, int renorm, int extra, float* __restrict__ extras) {
+                 int sigmoid, int renorm, int extra, float* __restrict__ extras, int group_best, float wscale) {
   extern __shared__ __align__(16) float smem[];
   int R = RC + extra;                              // rows of the matrix: the RC outputs that compete, then the extra ones
   float* rows = smem;                              // [kRouteTokens][kRouteChunk]
@@ -161,7 +163,7 @@ moe_route_kernel(const T* __restrict__ h, long long ldh, const float* __restrict
     for (int e = lane; e < R; e += 32) {
       const float logit = zt[e];
       zt[e] = 1.f / (1.f + expf(-logit));
-      pt[e] = correction != nullptr ? zt[e] + correction[e] : logit;
+      pt[e] = correction != nullptr ? zt[e] + correction[e] : group_best > 1 ? zt[e] : logit;
     }
   } else {
     float top_z = -INFINITY;
@@ -179,15 +181,28 @@ moe_route_kernel(const T* __restrict__ h, long long ldh, const float* __restrict
     for (int e = lane; e < R; e += 32) {
       zt[e] *= inv;
       if (correction != nullptr) pt[e] = zt[e] + correction[e];
+      else if (group_best > 1) pt[e] = zt[e];
     }
   }
   __syncwarp();
   const int size = R / groups;
   if (groups > 1 && keep < groups) {
     for (int g = lane; g < groups; g += 32) {
-      float best = -INFINITY;
-      for (int e = g * size; e < (g + 1) * size; ++e) best = fmaxf(best, pt[e]);
-      gt[g] = best;
+      float sum = 0.f, taken = INFINITY;
+      int at = -1;  // the last that was added, and its value: the next one is the largest behind it (ties: by index)
+      for (int b = 0; b < min(group_best, size); ++b) {
+        float best = -INFINITY;
+        int next = -1;
+        for (int e = g * size; e < (g + 1) * size; ++e) {
+          const float v = pt[e];
+          if ((v < taken || (v == taken && e > at)) && (next < 0 || v > best)) { best = v; next = e; }
+        }
+        if (next < 0) break;
+        sum += best;
+        taken = best;
+        at = next;
+      }
+      gt[g] = sum;
     }
     __syncwarp();
     // a group stays iff fewer than `keep` groups beat it (a tie goes to the lower index)
@@ -214,14 +229,14 @@ moe_route_kernel(const T* __restrict__ h, long long ldh, const float* __restrict
     if (at == 0x7fffffff) at = 0;  // fewer choosable outputs than `top`: cannot happen for a valid configuration
     if (lane == 0) {
       chosen[(size_t)n * top + k] = at;
-      weights[(size_t)n * top + k] = zt[at];
+      weights[(size_t)n * top + k] = renorm ? zt[at] : zt[at] * wscale;
       pt[at] = -INFINITY;
     }
     total += zt[at];
     __syncwarp();
   }
   if (lane == 0 && renorm) {
-    const float norm = 1.f / (total + 1e-20f);
+    const float norm = wscale / (total + 1e-20f);
     for (int k = 0; k < top; ++k) weights[(size_t)n * top + k] *= norm;
   }
 }
@@ -288,7 +303,7 @@ moe_gate_up_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__
 
 // One warp per (token, output channel c): the weighted sum over the token's chosen outputs. With `x` the sum does not
 // go to `out` but into the residual stream: x += mult * (ls_a * a + ls_b * sum), the update of a block whose mixer's
-// result a and feed-forward meet the stream together (a null scale is all ones). Null weights: every weight is one.
+// result a and feed-forward meet the stream together (a null scale is all ones; a null a: none). Null weights: every weight is one.
 // shared (or null): float32 [N, C] added to the sum, times shared_gate[n * ldsg] where that is given.
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -330,7 +345,7 @@ moe_down_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w_
       if (shared != nullptr) total = fmaf(shared_gate != nullptr ? shared_gate[(size_t)n * ldsg] : 1.f, shared[(size_t)n * C + c], total);
       if (x != nullptr) {
         const size_t at = (size_t)n * C + c;
-        x[at] = fmaf(mult, fmaf(ls_b ? ls_b[c] : 1.f, total, (ls_a ? ls_a[c] : 1.f) * a_res[at]), x[at]);
+        x[at] = fmaf(mult, fmaf(ls_b ? ls_b[c] : 1.f, total, a_res ? (ls_a ? ls_a[c] : 1.f) * a_res[at] : 0.f), x[at]);
       } else {
         out[(size_t)n * C + c] = total;
       }
@@ -343,9 +358,9 @@ moe_down_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w_
 // R: the outputs that compete; the matrix has R + extra rows.
 AKAS_API int akas_moe_route(const void* h, long long ldh, const float* w, const float* correction, int* chosen, float* weights,
                             int N, int C, int R, int groups, int keep, int top, int dtype, int sigmoid, int renorm, int extra,
-                            float* extras, cudaStream_t stream) {
+                            float* extras, int group_best, float wscale, cudaStream_t stream) {
   if (N <= 0) return 0;
-  if (R <= 0 || groups <= 0 || R % groups || keep <= 0 || keep > groups || top <= 0 || top > keep * (R / groups) || extra < 0 ||
+  if (R <= 0 || groups <= 0 || R % groups || keep <= 0 || keep > groups || top <= 0 || top > keep * (R / groups) || extra < 0 || group_best < 1 ||
       (extra > 0 && extras == nullptr))
     return (int)cudaErrorInvalidValue;
   const size_t smem = sizeof(float) * ((size_t)kRouteTokens * kRouteChunk + 2 * (size_t)kRouteTokens * (R + extra) + (size_t)kRouteTokens * groups +
@@ -365,9 +380,9 @@ AKAS_API int akas_moe_route(const void* h, long long ldh, const float* w, const 
   }
   if (dtype == AKAS_F32)
     return launch_ordinary(moe_route_kernel<float>, grid, dim3(kRouteTokens * 32), smem, stream, (const float*)h, ldh, w,
-                           correction, chosen, weights, N, C, R, groups, keep, top, sigmoid, renorm, extra, extras);
+                           correction, chosen, weights, N, C, R, groups, keep, top, sigmoid, renorm, extra, extras, group_best, wscale);
   return launch_ordinary(moe_route_kernel<bf16>, grid, dim3(kRouteTokens * 32), smem, stream, (const bf16*)h, ldh, w, correction,
-                         chosen, weights, N, C, R, groups, keep, top, sigmoid, renorm, extra, extras);
+                         chosen, weights, N, C, R, groups, keep, top, sigmoid, renorm, extra, extras, group_best, wscale);
 }
 
 AKAS_API int akas_moe_gate_up(const void* h, long long ldh, const void* w_gate_up, const int* chosen, void* act, int N,

@@ -123,7 +123,7 @@ __global__ void moe_combine_kernel(const bf16* __restrict__ h, long long ldh, co
     if (x != nullptr) {
       const float4 one = make_float4(1.f, 1.f, 1.f, 1.f);
       const float4 la = ls_a ? *reinterpret_cast<const float4*>(ls_a + c) : one, lb = ls_b ? *reinterpret_cast<const float4*>(ls_b + c) : one;
-      const float4 av = *reinterpret_cast<const float4*>(a_res + (size_t)n * C + c);
+      const float4 av = a_res ? *reinterpret_cast<const float4*>(a_res + (size_t)n * C + c) : make_float4(0.f, 0.f, 0.f, 0.f);
       float4 xv = *reinterpret_cast<float4*>(x + (size_t)n * C + c);
       xv.x = fmaf(mult, fmaf(lb.x, total.x, la.x * av.x), xv.x); xv.y = fmaf(mult, fmaf(lb.y, total.y, la.y * av.y), xv.y);
       xv.z = fmaf(mult, fmaf(lb.z, total.z, la.z * av.z), xv.z); xv.w = fmaf(mult, fmaf(lb.w, total.w, la.w * av.w), xv.w);

@@ -1,4 +1,5 @@
-// Mixers with a matrix state per head: gated linear attention and the gated delta rule, and what stands around
+// Mixers with a matrix state per head: gated linear attention (with keys, or with a forget gate that stands in for them)
+// and the gated delta rule, and what stands around
 // their recurrences (low-rank decay gates, a causal depthwise convolution with silu, unit-length q and k, the
 // step sizes and decays of the delta rule, the gated RMS norm of the read-out).
 //
@@ -62,6 +63,11 @@ __global__ void decay_gates_kernel(const T* __restrict__ low, long long ld, cons
 //   GLA:    s <- alpha_t[kk] s + k_t[kk] v_t[j];                                  o_t[j] = sum_kk s q_t[kk]
 //   FIXED:  the same with one constant decay per head in place of alpha_t[kk] (decay [H]); with `act`, q, k and v
 //           pass silu on their way in (the mixer's activations, applied in float32).
+//   GATE:   s <- g_t[kk] s + (1 - g_t[kk]) v_t[j], o_t[j] = sum_kk s silu(q_t[kk]), with the forget gate of a key channel
+//           g = low + (1 - low) sigmoid(z + b) from its logit z (k's place) and b, low [H * D] (decay's and beta's place);
+//           1 - g is computed as (1 - low) sigmoid(-(z + b)), which keeps its digits where the gate is nearly open. PART 1:
+//           a chunk's walk from an empty state, which leaves the state and the products of the gates per key channel in
+//           scratch, no outputs; PART 2: a chunk's walk from the state that scratch holds for its start, outputs only.
 //   DELTA:  s <- g_t s; u = beta_t (v_t[j] - sum_kk s k_t[kk]); s <- s + k_t[kk] u; o_t[j] = sum_kk s q_t[kk]
 constexpr int kPad = 4;  // floats between the R-blocks of a shared row: neighbouring lanes' 16-byte reads miss each other's banks
 
@@ -71,13 +77,34 @@ template <int KS> __device__ __forceinline__ float group_sum(float v) {
   return v;
 }
 
-template <typename T, int R, int KS, int CH, int TH, bool DELTA, bool FIXED = false>
+constexpr int kChunk = 64;  // tokens of a chunk of the recurrences that run in chunks
+
+// which (request, chunk of it) the block's chunk number is; false if there is none
+__device__ __forceinline__ bool find_chunk(const int* __restrict__ cu_seqlens, const int* __restrict__ slots, int R, int id,
+                                           int& req, int& first, int& len, int& index) {
+  for (int r = 0; r < R; ++r) {
+    const int b = cu_seqlens[r], e = cu_seqlens[r + 1];
+    const int chunks = slots[r] < 0 ? 0 : (e - b + kChunk - 1) / kChunk;
+    if (id < chunks) {
+      req = r; index = id; first = b + id * kChunk; len = min(kChunk, e - first);
+      return true;
+    }
+    id -= chunks;
+  }
+  return false;
+}
+
+enum { RULE_GLA = 0, RULE_DELTA = 1, RULE_FIXED = 2, RULE_GATE = 3 };
+
+template <typename T, int R, int KS, int CH, int TH, int RULE, int PART = 0>
 __global__ void __launch_bounds__(TH)
 scan_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ k, long long ldk, const T* __restrict__ v,
             long long ldv, const float* __restrict__ decay /* GLA: alpha [N, H * D]; DELTA: g [N, H] */,
             const float* __restrict__ beta /* DELTA: [N, H] */, float* __restrict__ state, long long slot_stride,
             const int* __restrict__ cu_seqlens, const int* __restrict__ slots, float* __restrict__ out, int H, int rep,
-            int D, int V, float q_scale, int write, int act) {
+            int D, int V, float q_scale, int write, int act, float* __restrict__ scratch, float* __restrict__ gates, int requests) {
+  constexpr bool DELTA = RULE == RULE_DELTA, FIXED = RULE == RULE_FIXED, GATE = RULE == RULE_GATE;
+  static_assert(PART == 0 || GATE, "only the forget gate's recurrence is walked in chunks");
   constexpr int VT = TH / KS;           // value channels of a block
   constexpr int ROW = KS * (R + kPad);  // floats of a padded shared row of key channels
   __shared__ __align__(16) float sq[CH][ROW];
@@ -86,10 +113,17 @@ scan_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ k, lon
   __shared__ float sv[CH][VT];
   __shared__ float sg[CH], sb[CH];
 
-  const int h = blockIdx.x, req = blockIdx.y;
+  const int h = blockIdx.x;
+  int req = blockIdx.y, t_begin, t_end;
+  if (PART == 0) {
+    t_begin = cu_seqlens[req], t_end = cu_seqlens[req + 1];
+    if (slots[req] < 0 || t_end <= t_begin) return;
+  } else {
+    int len, index;
+    if (!find_chunk(cu_seqlens, slots, requests, blockIdx.y, req, t_begin, len, index)) return;
+    t_end = t_begin + len;
+  }
   const int slot = slots[req];
-  const int t_begin = cu_seqlens[req], t_end = cu_seqlens[req + 1];
-  if (slot < 0 || t_end <= t_begin) return;
   const int ks = threadIdx.x % KS, jl = threadIdx.x / KS;
   const int j = blockIdx.z * VT + jl;
   const bool live = j < V;
@@ -97,11 +131,16 @@ scan_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ k, lon
   const int kk0 = ks * R;
 
   float s[R];
-  float* srow = state + (size_t)slot * slot_stride + ((size_t)h * V + (live ? j : 0)) * D;
-  const bool vec = D % 4 == 0 && slot_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(state) & 15) == 0;
+  float* srow = (PART == 0 ? state + (size_t)slot * slot_stride : scratch + (size_t)blockIdx.y * H * V * D) + ((size_t)h * V + (live ? j : 0)) * D;
+  const bool vec = D % 4 == 0 && (PART != 0 || slot_stride % 4 == 0) && (reinterpret_cast<uintptr_t>(PART == 0 ? state : scratch) & 15) == 0;
+  float kept[PART == 1 ? R : 1];  // the products of the gates so far
+#pragma unroll
+  for (int r = 0; r < (PART == 1 ? R : 1); ++r) kept[r] = 1.f;
 #pragma unroll
   for (int r = 0; r < R; r += 4) {
-    if (live && vec && kk0 + r + 3 < D) {
+    if (PART == 1) {
+      s[r] = s[r + 1] = s[r + 2] = s[r + 3] = 0.f;
+    } else if (live && vec && kk0 + r + 3 < D) {
       const float4 x = *reinterpret_cast<const float4*>(srow + kk0 + r);
       s[r] = x.x; s[r + 1] = x.y; s[r + 2] = x.z; s[r + 3] = x.w;
     } else {
@@ -114,7 +153,7 @@ scan_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ k, lon
   // when that is done: the recurrence never waits for global memory except at its first chunk.
   constexpr int NQ = (CH * KS * R + TH - 1) / TH, NV = (CH * VT + TH - 1) / TH;
   T rq[NQ], rk[NQ], rv[NV];  // as fetched: widening them here would make the loop below wait for the loads at once
-  float ra[DELTA || FIXED ? 1 : NQ], rg = 0.f, rb = 0.f;
+  float ra[RULE == RULE_GLA ? NQ : 1], rg = 0.f, rb = 0.f;
   const float fixed = FIXED ? decay[h] : 0.f;
   const T zero = from_f32<T>(0.f);
   auto fetch = [&](int c0) {
@@ -125,9 +164,9 @@ scan_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ k, lon
       const int t = i / (KS * R), kk = i % (KS * R);
       const bool in = t < count && kk < D;
       const size_t n = (size_t)(c0 + t);
-      rq[u] = in ? q[n * ldq + (size_t)hk * D + kk] : zero;
+      if (PART != 1) rq[u] = in ? q[n * ldq + (size_t)hk * D + kk] : zero;
       rk[u] = in ? k[n * ldk + (size_t)hk * D + kk] : zero;
-      if (!DELTA && !FIXED) ra[u] = in ? decay[n * ((size_t)H * D) + (size_t)h * D + kk] : 0.f;
+      if (RULE == RULE_GLA) ra[u] = in ? decay[n * ((size_t)H * D) + (size_t)h * D + kk] : 0.f;
     }
 #pragma unroll
     for (int u = 0; u < NV; ++u) {
@@ -150,11 +189,17 @@ scan_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ k, lon
       if (i < CH * KS * R) {
         const int t = i / (KS * R), kk = i % (KS * R);
         const int at = kk + (kk / R) * kPad;
-        float qv = to_f32(rq[u]), kv = to_f32(rk[u]);
+        float qv = PART != 1 ? to_f32(rq[u]) : 0.f, kv = to_f32(rk[u]);
         if (FIXED && act) { qv *= sigmoid_f(qv); kv *= sigmoid_f(kv); }
-        sq[t][at] = qv * q_scale;
+        if (GATE) {
+          const float low = kk < D ? beta[(size_t)h * D + kk] : 1.f, z = kk < D ? kv + decay[(size_t)h * D + kk] : 0.f;
+          qv *= sigmoid_f(qv);
+          kv = (1.f - low) * sigmoid_f(-z);
+          sa[t][at] = fmaf(1.f - low, sigmoid_f(z), low);
+        }
+        if (PART != 1) sq[t][at] = qv * q_scale;
         sk[t][at] = kv;
-        if (!DELTA && !FIXED) sa[t][at] = ra[u];
+        if (RULE == RULE_GLA) sa[t][at] = ra[u];
       }
     }
 #pragma unroll
@@ -211,18 +256,31 @@ scan_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ k, lon
 #pragma unroll
         for (int r = 0; r < R; r += 4) {
           const float4 kv = *reinterpret_cast<const float4*>(kr + r);
-          const float4 qv = *reinterpret_cast<const float4*>(qr + r);
           const float4 av = *reinterpret_cast<const float4*>(ar + r);
           s[r] = fmaf(av.x, s[r], kv.x * vj); s[r + 1] = fmaf(av.y, s[r + 1], kv.y * vj);
           s[r + 2] = fmaf(av.z, s[r + 2], kv.z * vj); s[r + 3] = fmaf(av.w, s[r + 3], kv.w * vj);
+          if (PART == 1) {
+            if (threadIdx.x < 32 && blockIdx.z == 0) {  // one warp holds every key channel's product
+              kept[r] *= av.x; kept[r + 1] *= av.y; kept[r + 2] *= av.z; kept[r + 3] *= av.w;
+            }
+            continue;
+          }
+          const float4 qv = *reinterpret_cast<const float4*>(qr + r);
           acc = fmaf(s[r], qv.x, acc); acc2 = fmaf(s[r + 1], qv.y, acc2); acc = fmaf(s[r + 2], qv.z, acc); acc2 = fmaf(s[r + 3], qv.w, acc2);
         }
       }
+      if (PART == 1) continue;
       acc = group_sum<KS>(acc + acc2);
       if (ks == 0 && live) out[(size_t)(c0 + t) * ((size_t)H * V) + (size_t)h * V + j] = acc;
     }
   }
-  if (write && live) {
+  if (PART == 1 && blockIdx.z == 0 && jl == 0) {
+    float* grow = gates + ((size_t)blockIdx.y * H + h) * D;
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (kk0 + r < D) grow[kk0 + r] = kept[r];
+  }
+  if ((PART == 0 ? write != 0 : PART == 1) && live) {
 #pragma unroll
     for (int r = 0; r < R; r += 4) {
       if (vec && kk0 + r + 3 < D) {
@@ -236,12 +294,14 @@ scan_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ k, lon
   }
 }
 
-template <typename T, bool DELTA, bool FIXED = false>
+template <typename T, int RULE, int PART = 0>
 int launch_scan(const T* q, long long ldq, const T* k, long long ldk, const T* v, long long ldv, const float* decay,
                 const float* beta, float* state, long long slot_stride, const int* cu_seqlens, const int* slots, float* out,
                 int tokens, int requests, int H, int rep, int D, int V, float q_scale, int write, cudaStream_t stream,
-                int act = 0) {
+                int act = 0, float* scratch = nullptr, float* gates = nullptr, int chunks = 0) {
   if (requests <= 0 || H <= 0) return 0;
+  const int walks = PART == 0 ? requests : chunks;  // what the blocks of one head and tile of value channels walk each
+  if (walks > 65535) return (int)cudaErrorInvalidValue;
   if (D > 1024) return (int)cudaErrorInvalidValue;
   // (Blocks of 64 threads, which spread a head's value channels over four times as many SMs when a step holds few
   // long portions, were measured and dropped: a token's cost is the latency of its chain of shared-memory reads, sums
@@ -249,15 +309,17 @@ int launch_scan(const T* q, long long ldq, const T* k, long long ldk, const T* v
   (void)tokens;
 #define AKAS_SCAN(R, KS, CH)                                                                                              \
   {                                                                                                                       \
-    const dim3 grid(H, requests, (V + 256 / KS - 1) / (256 / KS));                                                        \
-    return launch_ordinary(scan_kernel<T, R, KS, CH, 256, DELTA, FIXED>, grid, dim3(256), 0, stream, q, ldq, k, ldk, v, ldv,  \
-                          decay, beta, state, slot_stride, cu_seqlens, slots, out, H, rep, D, V, q_scale, write, act);    \
+    const dim3 grid(H, walks, (V + 256 / KS - 1) / (256 / KS));                                                           \
+    return launch_ordinary(scan_kernel<T, R, KS, CH, 256, RULE, PART>, grid, dim3(256), 0, stream, q, ldq, k, ldk, v, ldv,   \
+                          decay, beta, state, slot_stride, cu_seqlens, slots, out, H, rep, D, V, q_scale, write, act,     \
+                          scratch, gates, requests);                                                                      \
   }
   if (D <= 8) AKAS_SCAN(8, 1, 16)
   if (D <= 16) AKAS_SCAN(8, 2, 16)
   if (D <= 32) AKAS_SCAN(8, 4, 16)
   if (D <= 64) AKAS_SCAN(16, 4, 16)
   if (D <= 128) AKAS_SCAN(16, 8, 16)
+  if (PART != 0) return (int)cudaErrorInvalidValue;  // (the caller walks larger keys token by token)
   if (D <= 256) AKAS_SCAN(16, 16, 8)
   if (D <= 512) AKAS_SCAN(16, 32, 4)
   AKAS_SCAN(32, 32, 2)
@@ -276,22 +338,7 @@ int launch_scan(const T* q, long long ldq, const T* k, long long ldk, const T* v
 // Everything is float32 fused multiply-adds (the decays' powers come from a float64 pow, rounded once); sums run in
 // a fixed order that depends on where a chunk starts in the step, so a result differs from the token-by-token
 // kernel's, and between ways of cutting a prompt, by rounding only. Key sizes up to kChunkMaxD.
-constexpr int kChunk = 64, kChunkVT = 64, kChunkMaxD = 128, kChunkThreads = 256;
-
-// which (request, chunk of it) the block's chunk number is; false if there is none
-__device__ __forceinline__ bool find_chunk(const int* __restrict__ cu_seqlens, const int* __restrict__ slots, int R, int id,
-                                           int& req, int& first, int& len, int& index) {
-  for (int r = 0; r < R; ++r) {
-    const int b = cu_seqlens[r], e = cu_seqlens[r + 1];
-    const int chunks = slots[r] < 0 ? 0 : (e - b + kChunk - 1) / kChunk;
-    if (id < chunks) {
-      req = r; index = id; first = b + id * kChunk; len = min(kChunk, e - first);
-      return true;
-    }
-    id -= chunks;
-  }
-  return false;
-}
+constexpr int kChunkVT = 64, kChunkMaxD = 128, kChunkThreads = 256;
 
 // Stages `live` rows of `cols` channels (src row pitch ld) into shared memory rows of `pitch` floats as float32, silu'd
 // where `act`, times `scale` or, where `pw` is given, times pw[live - 1 - row]; rows from `live` to `rows` and the columns
@@ -529,6 +576,45 @@ int launch_chunks(const T* q, long long ldq, const T* k, long long ldk, const T*
                          cu_seqlens, slots, (const float*)scratch, out, requests, H, D, V, DP, q_scale, act);
 }
 
+// ------------------------------------------------------------------------------------------------ forget gates, in chunks
+//
+// The recurrence whose forget gate also writes, for prompt portions: every chunk of kChunk tokens is walked from an empty
+// state at once (scan_kernel, PART 1), gate_carry puts the chunks' ends together, S_(j+1) = diag(product of chunk j's
+// gates) S_j + U_j, leaving every chunk's start where its end stood and the last one in the slot, and every chunk is
+// walked again from its start (PART 2), for its outputs. No quotient of gate products is ever formed, so gates near zero
+// cost no digits; a result differs from the walk token by token, and between ways of cutting a prompt, by rounding only.
+__global__ void gate_carry_kernel(const float* __restrict__ gates, float* __restrict__ state, long long slot_stride,
+                                  const int* __restrict__ cu_seqlens, const int* __restrict__ slots, float* __restrict__ scratch,
+                                  int H, int D, int V, int write) {
+  const int req = blockIdx.x, h = blockIdx.y;
+  const int slot = slots[req];
+  if (slot < 0) return;
+  int base = 0;  // the number of the request's first chunk
+  for (int r = 0; r < req; ++r) base += slots[r] < 0 ? 0 : (cu_seqlens[r + 1] - cu_seqlens[r] + kChunk - 1) / kChunk;
+  const int chunks = (cu_seqlens[req + 1] - cu_seqlens[req] + kChunk - 1) / kChunk;
+  float* srow = state + (size_t)slot * slot_stride + (size_t)h * V * D;
+  for (int i = blockIdx.z * blockDim.x + threadIdx.x; i < V * D; i += gridDim.z * blockDim.x) {
+    float s = srow[i];
+    for (int j0 = 0; j0 < chunks; j0 += 8) {  // eight chunks' sums are fetched at once: the chain itself waits for no load
+      float add[8], keep[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const size_t at = (size_t)(base + j0 + e) * H + h;
+        add[e] = j0 + e < chunks ? scratch[at * V * D + i] : 0.f;
+        keep[e] = j0 + e < chunks ? gates[at * D + i % D] : 0.f;
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        if (j0 + e < chunks) {
+          scratch[((size_t)(base + j0 + e) * H + h) * V * D + i] = s;
+          s = fmaf(keep[e], s, add[e]);
+        }
+      }
+    }
+    if (write && chunks > 0) srow[i] = s;
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ causal convolution
 //
 // y[n, c] = silu(sum_j taps[c, j] * x_(i - L + 1 + j)) for the i-th token of its request in this step; inputs before
@@ -646,7 +732,7 @@ __global__ void delta_prep_kernel(float* __restrict__ y, long long ldy, int G, i
 //
 // One warp per (token, head): out = o / sqrt(mean(o^2) + eps) * w * f(gate) * out_scale, f = silu or (sigmoid != 0)
 // the sigmoid alone; the output's rows have a pitch of their own. A norm over all heads together is the call with one
-// head of H * V channels. w may be null: the division alone, every weight one.
+// head of H * V channels. w may be null: the division alone, every weight one; gate may be null: no gate.
 __device__ __forceinline__ float4 norm_weight4(const float* __restrict__ w, int j) {
   return w != nullptr ? *reinterpret_cast<const float4*>(w + j) : make_float4(1.f, 1.f, 1.f, 1.f);
 }
@@ -675,7 +761,7 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const float* _
         if (j < V) {
           x[i] = *reinterpret_cast<const float4*>(row + j);
           wv[i] = norm_weight4(w, j);
-          load4(gate + (size_t)n * ldg + (size_t)h * V + j, gv[i]);
+          if (gate != nullptr) load4(gate + (size_t)n * ldg + (size_t)h * V + j, gv[i]);
           ss = fmaf(x[i].x, x[i].x, ss); ss = fmaf(x[i].y, x[i].y, ss); ss = fmaf(x[i].z, x[i].z, ss); ss = fmaf(x[i].w, x[i].w, ss);
         }
       }
@@ -686,7 +772,7 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const float* _
         const int j = lane * 4 + i * 128;
         if (j < V) {
 #pragma unroll
-          for (int e = 0; e < 4; ++e) gv[i][e] = sigmoid ? sigmoid_f(gv[i][e]) : gv[i][e] * sigmoid_f(gv[i][e]);
+          for (int e = 0; e < 4; ++e) gv[i][e] = gate == nullptr ? 1.f : sigmoid ? sigmoid_f(gv[i][e]) : gv[i][e] * sigmoid_f(gv[i][e]);
           const float r[4] = {x[i].x * inv * wv[i].x * gv[i][0], x[i].y * inv * wv[i].y * gv[i][1], x[i].z * inv * wv[i].z * gv[i][2],
                               x[i].w * inv * wv[i].w * gv[i][3]};
           TO* dst = out + (size_t)n * ldo + (size_t)h * V + j;
@@ -711,9 +797,9 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const float* _
       const float4 x = *reinterpret_cast<const float4*>(row + j);
       const float4 wv = norm_weight4(w, j);
       float gv[4];
-      load4(gate + (size_t)n * ldg + (size_t)h * V + j, gv);
+      if (gate != nullptr) load4(gate + (size_t)n * ldg + (size_t)h * V + j, gv);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) gv[e] = sigmoid ? sigmoid_f(gv[e]) : gv[e] * sigmoid_f(gv[e]);
+      for (int e = 0; e < 4; ++e) gv[e] = gate == nullptr ? 1.f : sigmoid ? sigmoid_f(gv[e]) : gv[e] * sigmoid_f(gv[e]);
       const float r[4] = {x.x * inv * wv.x * gv[0], x.y * inv * wv.y * gv[1], x.z * inv * wv.z * gv[2], x.w * inv * wv.w * gv[3]};
       TO* dst = out + (size_t)n * ldo + (size_t)h * V + j;
       if (sizeof(TO) == 4) {
@@ -729,8 +815,8 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const float* _
   ss = warp_sum(ss);
   const float inv = out_scale / sqrtf(ss / (float)V + eps);
   for (int j = lane; j < V; j += 32) {
-    const float gv = to_f32(gate[(size_t)n * ldg + (size_t)h * V + j]);
-    out[(size_t)n * ldo + (size_t)h * V + j] = from_f32<TO>(row[j] * inv * (w != nullptr ? w[j] : 1.f) * (sigmoid ? sigmoid_f(gv) : gv * sigmoid_f(gv)));
+    const float gv = gate != nullptr ? to_f32(gate[(size_t)n * ldg + (size_t)h * V + j]) : 0.f;
+    out[(size_t)n * ldo + (size_t)h * V + j] = from_f32<TO>(row[j] * inv * (w != nullptr ? w[j] : 1.f) * (gate == nullptr ? 1.f : sigmoid ? sigmoid_f(gv) : gv * sigmoid_f(gv)));
   }
 }
 
@@ -752,9 +838,9 @@ AKAS_API int akas_gla_scan(const void* q, long long ldq, const void* k, long lon
                            float* out, int tokens, int requests, int H, int D, int V, float q_scale, int write, int dtype,
                            cudaStream_t stream) {
   if (dtype == AKAS_F32)
-    return launch_scan<float, false>((const float*)q, ldq, (const float*)k, ldk, (const float*)v, ldv, alpha, nullptr, state,
+    return launch_scan<float, RULE_GLA>((const float*)q, ldq, (const float*)k, ldk, (const float*)v, ldv, alpha, nullptr, state,
                                      slot_stride, cu_seqlens, slots, out, tokens, requests, H, 1, D, V, q_scale, write, stream);
-  return launch_scan<bf16, false>((const bf16*)q, ldq, (const bf16*)k, ldk, (const bf16*)v, ldv, alpha, nullptr, state,
+  return launch_scan<bf16, RULE_GLA>((const bf16*)q, ldq, (const bf16*)k, ldk, (const bf16*)v, ldv, alpha, nullptr, state,
                                   slot_stride, cu_seqlens, slots, out, tokens, requests, H, 1, D, V, q_scale, write, stream);
 }
 
@@ -764,10 +850,10 @@ AKAS_API int akas_decay_scan(const void* q, long long ldq, const void* k, long l
                              float* out, int tokens, int requests, int H, int D, int V, float q_scale, int act, int write,
                              int dtype, cudaStream_t stream) {
   if (dtype == AKAS_F32)
-    return launch_scan<float, false, true>((const float*)q, ldq, (const float*)k, ldk, (const float*)v, ldv, decay, nullptr,
+    return launch_scan<float, RULE_FIXED>((const float*)q, ldq, (const float*)k, ldk, (const float*)v, ldv, decay, nullptr,
                                            state, slot_stride, cu_seqlens, slots, out, tokens, requests, H, 1, D, V, q_scale,
                                            write, stream, act);
-  return launch_scan<bf16, false, true>((const bf16*)q, ldq, (const bf16*)k, ldk, (const bf16*)v, ldv, decay, nullptr, state,
+  return launch_scan<bf16, RULE_FIXED>((const bf16*)q, ldq, (const bf16*)k, ldk, (const bf16*)v, ldv, decay, nullptr, state,
                                         slot_stride, cu_seqlens, slots, out, tokens, requests, H, 1, D, V, q_scale, write,
                                         stream, act);
 }
@@ -792,12 +878,46 @@ AKAS_API int akas_decay_scan_chunked(const void* q, long long ldq, const void* k
                        out, scratch, tokens, requests, H, D, V, q_scale, act, write, stream);
 }
 
+// The recurrence whose forget gate also writes (RULE_GATE above), token by token: f the gates' logits, f_bias and lower [H * D].
+AKAS_API int akas_gate_scan(const float* q, long long ldq, const float* f, long long ldf, const float* v, long long ldv,
+                            const float* f_bias, const float* lower, float* state, long long slot_stride, const int* cu_seqlens,
+                            const int* slots, float* out, int tokens, int requests, int H, int D, int V, int write,
+                            cudaStream_t stream) {
+  return launch_scan<float, RULE_GATE>(q, ldq, f, ldf, v, ldv, f_bias, lower, state, slot_stride, cu_seqlens, slots, out, tokens,
+                                       requests, H, 1, D, V, 1.f, write, stream);
+}
+
+// Floats of scratch that akas_gate_scan_chunked needs; 0 where it does not take the sizes (the token-by-token kernel does).
+AKAS_API long long akas_gate_chunk_scratch(int tokens, int requests, int H, int D, int V) {
+  const long long chunks = (tokens + kChunk - 1) / kChunk + requests;
+  if (D > kChunkMaxD || tokens <= 0 || requests <= 0 || chunks > 65535) return 0;
+  return chunks * H * D * (V + 1);
+}
+
+AKAS_API int akas_gate_scan_chunked(const float* q, long long ldq, const float* f, long long ldf, const float* v, long long ldv,
+                                    const float* f_bias, const float* lower, float* state, long long slot_stride,
+                                    const int* cu_seqlens, const int* slots, float* out, float* scratch, int tokens, int requests,
+                                    int H, int D, int V, int write, cudaStream_t stream) {
+  if (tokens <= 0 || requests <= 0 || H <= 0) return 0;
+  if (akas_gate_chunk_scratch(tokens, requests, H, D, V) == 0 || scratch == nullptr) return (int)cudaErrorInvalidValue;
+  const int chunks = (tokens + kChunk - 1) / kChunk + requests;  // at most: every request may end with a part of a chunk
+  float* gates = scratch + (size_t)chunks * H * D * V;
+  int err = launch_scan<float, RULE_GATE, 1>(q, ldq, f, ldf, v, ldv, f_bias, lower, state, slot_stride, cu_seqlens, slots, out, tokens,
+                                             requests, H, 1, D, V, 1.f, 1, stream, 0, scratch, gates, chunks);
+  if (err) return err;
+  err = launch_ordinary(gate_carry_kernel, dim3(requests, H, min(64, (V * D + 255) / 256)), dim3(256), 0, stream, (const float*)gates,
+                        state, slot_stride, cu_seqlens, slots, scratch, H, D, V, write);
+  if (err) return err;
+  return launch_scan<float, RULE_GATE, 2>(q, ldq, f, ldf, v, ldv, f_bias, lower, state, slot_stride, cu_seqlens, slots, out, tokens,
+                                          requests, H, 1, D, V, 1.f, 0, stream, 0, scratch, gates, chunks);
+}
+
 AKAS_API int akas_delta_scan(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv,
                              const float* beta, const float* g, float* state, long long slot_stride, const int* cu_seqlens,
                              const int* slots, float* out, int tokens, int requests, int H, int G, int D, int V, int write,
                              cudaStream_t stream) {
   if (G <= 0 || H % G) return (int)cudaErrorInvalidValue;
-  return launch_scan<float, true>(q, ldq, k, ldk, v, ldv, g, beta, state, slot_stride, cu_seqlens, slots, out, tokens,
+  return launch_scan<float, RULE_DELTA>(q, ldq, k, ldk, v, ldv, g, beta, state, slot_stride, cu_seqlens, slots, out, tokens,
                                   requests, H, H / G, D, V, 1.f, write, stream);
 }
 

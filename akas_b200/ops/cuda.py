@@ -30,6 +30,11 @@ launch_count = 0  # kernels launched through this module since import (library p
 _SIGNATURES = {
     "elementwise": {
         "akas_embedding": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+        "akas_bigram_embedding": [c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                                  c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+        "akas_depth_average": [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
+        "akas_depth_average_norm": [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_float, c_int,
+                                    c_void_p, c_int, c_void_p],
         "akas_rmsnorm": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p],
         "akas_rmsnorm_pair": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_void_p],
         "akas_round_rows": [c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p],
@@ -55,7 +60,7 @@ _SIGNATURES = {
     },
     "moe": {
         "akas_moe_route": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                           c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+                           c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_float, c_void_p],
         "akas_moe_gate_up": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                              c_void_p, c_int, c_void_p],
         "akas_moe_down": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
@@ -74,6 +79,12 @@ _SIGNATURES = {
                             c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "akas_gated_rmsnorm": [c_void_p, c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                c_int, c_float, c_longlong, c_void_p],
+        "akas_gate_scan": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_longlong,
+                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "akas_gate_chunk_scratch": [c_int, c_int, c_int, c_int, c_int],
+        "akas_gate_scan_chunked": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
+                                   c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                                   c_void_p],
         "akas_decay_chunk_scratch": [c_int, c_int, c_int, c_int, c_int],
         "akas_decay_scan_chunked": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong,
                                     c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
@@ -86,16 +97,19 @@ _SIGNATURES = {
         "akas_qk_norm_store": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_float,
                                c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p,
-                               c_void_p, c_int, c_void_p],
+                               c_void_p, c_int, c_float, c_int, c_void_p],
+        "akas_pool_blocks": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                             c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "akas_attention_general": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int,
                                    c_int, c_float, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_int,
-                                   c_int, c_int, c_int, c_void_p, c_float, c_longlong, c_longlong, c_int, c_int, c_void_p],
+                                   c_int, c_int, c_int, c_void_p, c_float, c_longlong, c_longlong, c_int, c_int, c_void_p, c_void_p,
+                                   c_void_p, c_int, c_int, c_int, c_void_p],
     },
     "attention_general_tc": {
         "akas_attention_general_tc": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float,
                                       c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_int,
                                       c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_longlong, c_void_p, c_int,
-                                      c_longlong, c_int, c_int, c_void_p],
+                                      c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "akas_attention_general_tc_takes": [c_int, c_int],
     },
     "moe_grouped": {
@@ -213,7 +227,7 @@ _SIGNATURES = {
     },
 }
 
-_RESTYPES = {"akas_decay_chunk_scratch": c_longlong}  # everything else returns an int (an error code or a small answer)
+_RESTYPES = {"akas_decay_chunk_scratch": c_longlong, "akas_gate_chunk_scratch": c_longlong}  # everything else returns an int (an error code or a small answer)
 _functions = {}
 
 
@@ -440,6 +454,55 @@ def embedding(token_ids, table):
 
 
 @_flushes
+def bigram_embedding(token_ids, table, pairs, mul_prev, mul_cur, state, cu_seqlens, seq_of_token, slots, out=None):
+    """The embedding's row of every token plus the row of ``pairs`` [buckets + 1, C] that the token in front of it and the
+    token pick. ``state`` int32 [slots, 1]; ``out`` float32 [2, N, C]: both halves receive the result."""
+    n, c = token_ids.numel(), table.shape[1]
+    if pairs.dtype != table.dtype or pairs.shape[1] != c:
+        raise ValueError("bigram_embedding takes two tables of one dtype and width")
+    if state.dtype != torch.int32 or state.shape[1] != 1 or state.stride(0) != 1:
+        raise ValueError("bigram_embedding keeps one int32 per slot")
+    if out is None:
+        first, both = torch.empty((n, c), dtype=torch.float32, device=table.device), None
+    else:
+        if out.dtype != torch.float32 or out.shape != (2, n, c) or not out.is_contiguous():
+            raise ValueError("bigram_embedding writes to dense float32 [2, N, C]")
+        first, both = out[0], out[1]
+    _check(_fn("elementwise", "akas_bigram_embedding")(
+        _ptr(token_ids), _ptr(_dense(table, "table")), _ptr(_dense(pairs, "pairs")), int(mul_prev), int(mul_cur), pairs.shape[0] - 1,
+        _ptr(state), _ptr(cu_seqlens), _ptr(seq_of_token), _ptr(slots), _ptr(first), _ptr(both), n, c, _code(table), _stream()),
+        "bigram_embedding")
+    return first if both is None else both
+
+
+@_flushes
+def depth_average(history, count, weights, out, rows=None, norm=None):
+    """sum_j weights[j] * history[j] over j < count for dense float32 history [.., N, C] (``rows``: of those rows alone).
+    ``norm`` = (weight, eps, zero_centered, dtype): where the product behind that RMSNorm would not compute it on its way
+    in, the same pass makes it. Returns (result, normed result or None)."""
+    _, n, c = history.shape
+    if history.dtype != torch.float32 or not history.is_contiguous() or weights.dtype != torch.float32 or weights.numel() != count:
+        raise ValueError("depth_average takes dense float32 history [.., N, C] and one float32 weight per summand")
+    m = rows.numel() if rows is not None else n
+    if out is None:
+        out = torch.empty((m, c), dtype=torch.float32, device=history.device)
+    elif out.dtype != torch.float32 or out.shape != (m, c) or not out.is_contiguous():
+        raise ValueError("depth_average writes to dense float32 rows")
+    args = (_ptr(history), n * c, count, _ptr(weights), _ptr(out), _ptr(rows), m, c)
+    if norm is not None:
+        weight, eps, zero_centered, dtype = norm
+        if dtype == torch.float32 or not (decode_products == "stream" or _skinny_fits(m, c)):
+            y = torch.empty((m, c), dtype=dtype, device=history.device)
+            err = _fn("elementwise", "akas_depth_average_norm")(*args, _ptr(weight), float(eps), int(bool(zero_centered)), _ptr(y),
+                                                               _CODE[dtype], _stream())
+            if err != 3999:
+                _check(err, "depth_average with a norm")
+                return out, y
+    _check(_fn("elementwise", "akas_depth_average")(*args, _stream()), "depth_average")
+    return out, None
+
+
+@_flushes
 def take_tokens(token_ids, source, previous):
     """token_ids[i] = previous[source[i]] where source[i] >= 0 (all int32, in place)."""
     _check(_fn("elementwise", "akas_take_tokens")(_ptr(token_ids), _ptr(source), _ptr(previous), previous.numel(),
@@ -523,7 +586,7 @@ def scale_cap(x, scale=1.0, cap=0.0):
 def zero_rows(state, slot):
     """state[:, slot] = 0 for a contiguous tensor [layers, slots, ...]."""
     row = state[0, 0].numel()
-    if state.dtype != torch.float32 or not state.is_contiguous():
+    if state.dtype not in (torch.float32, torch.int32) or not state.is_contiguous():  # (four bytes of zeros are zero in both)
         state[:, slot].zero_()
         return
     _check(_fn("elementwise", "akas_zero_row")(_ptr(state), row, int(slot), state.shape[0], state[0].numel(), _stream()),
@@ -1446,6 +1509,29 @@ def gla_scan(q, k, v, alpha, state, cu_seqlens, slots, heads, dim, vdim, q_scale
 
 
 @_flushes
+def hgrn2_scan(q, f, v, f_bias, lower, state, cu_seqlens, slots, heads, dim, vdim, write=True, longest=None):
+    """The recurrence whose forget gate also writes, on float32 rows of a product. In chunks (three kernels, see
+    csrc/recurrent.cu) when some request of the step brings at least _GATE_CHUNKED_FROM tokens (``longest``) and the key
+    size allows, token by token otherwise."""
+    n = q.shape[0]
+    if any(t.dtype != torch.float32 for t in (q, f, v, f_bias, lower)) or f_bias.numel() != heads * dim or lower.numel() != heads * dim:
+        raise ValueError("hgrn2_scan takes float32 inputs and one bias and lower bound per key channel")
+    (qp, ldq), (fp, ldf), (vp, ldv) = _rows(q, "q"), _rows(f, "f"), _rows(v, "v")
+    sp, stride = _slot_rows(state, "state")
+    out = torch.empty((n, heads * vdim), dtype=torch.float32, device=q.device)
+    head = (qp, ldq, fp, ldf, vp, ldv, _ptr(f_bias), _ptr(lower), sp, stride, _ptr(cu_seqlens), _ptr(slots), _ptr(out))
+    tail = (n, slots.numel(), heads, dim, vdim, int(bool(write)), _stream())
+    if decay_scan_kernels == "auto" and longest is not None and longest >= _GATE_CHUNKED_FROM:
+        words = int(_fn("recurrent", "akas_gate_chunk_scratch")(n, slots.numel(), heads, dim, vdim))
+        if words:
+            scratch = torch.empty(words, dtype=torch.float32, device=q.device)
+            _check(_fn("recurrent", "akas_gate_scan_chunked")(*head, _ptr(scratch), *tail), "hgrn2_scan (chunks)", kernels=3)
+            return out
+    _check(_fn("recurrent", "akas_gate_scan")(*head, *tail), "hgrn2_scan")
+    return out
+
+
+@_flushes
 def causal_conv_silu(x, taps, state, cu_seqlens, seq_of_token, slots, write=True):
     n, c = x.shape
     l = taps.shape[1]
@@ -1499,14 +1585,14 @@ def gated_rmsnorm(o, weight, eps, gate, heads, vdim, out_dtype, gate_activation=
         raise ValueError(f"unknown gate activation {gate_activation!r}")
     if weight is not None and (weight.dtype != torch.float32 or weight.numel() != vdim):
         raise ValueError("gated_rmsnorm: the weight is float32 [vdim] (None: the division alone)")
-    gp, ldg = _rows(gate, "gate")
+    gp, ldg = _rows(gate, "gate") if gate is not None else (None, 0)
     if out is None:
         out = torch.empty((n, heads * vdim), dtype=out_dtype, device=o.device)
     elif out.shape != (n, heads * vdim):
         raise ValueError("gated_rmsnorm: out must be [N, heads * vdim]")
     op, ldo = _rows(out, "out")
     _check(_fn("recurrent", "akas_gated_rmsnorm")(_ptr(o), _ptr(weight), float(eps), gp, ldg, op, n, heads, vdim,
-                                                 _code(gate), _code(out), int(gate_activation == "sigmoid"),
+                                                 _code(out if gate is None else gate), _code(out), int(gate_activation == "sigmoid"),
                                                  float(out_scale), ldo, _stream()), "gated_rmsnorm")
     return out
 
@@ -1518,6 +1604,7 @@ decay_scan_kernels = os.environ.get("AKAS_B200_DECAY_SCAN", "auto")
 if decay_scan_kernels not in ("auto", "tokens"):
     raise ValueError(f"AKAS_B200_DECAY_SCAN must be auto or tokens, got {decay_scan_kernels!r}")
 _CHUNKED_FROM = 48
+_GATE_CHUNKED_FROM = 160  # the forget gates' recurrence walks every chunk twice: it pays from three chunks on
 
 
 @_flushes
@@ -1552,8 +1639,11 @@ def decay_scan(q, k, v, decay, state, cu_seqlens, slots, heads, dim, vdim, q_sca
 @_flushes
 def qk_norm_store(q, k, v, heads, kv_heads, dim, vdim, q_weight, k_weight, eps, k_pool, v_pool, block_table,
                   seq_of_token, positions, page_size, write=True, cos=None, sin=None, interleaved=False,
-                  q_bias=None, k_bias=None, v_bias=None, unit_eps=None):
+                  q_bias=None, k_bias=None, v_bias=None, unit_eps=None, temperature=None):
     n = q.shape[0]
+    coef, every = (0.0, 0) if temperature is None else temperature
+    if temperature is not None and (int(every) != every or every < 1):
+        raise ValueError("qk_norm_store: a temperature grows every whole number of positions")
     if not (q.dtype == k.dtype == v.dtype) or k_pool.dtype != v_pool.dtype:
         raise TypeError("qk_norm_store: q, k, v must have one dtype, and so must the pages")
     if q.dtype != k_pool.dtype and q.dtype != torch.float32:
@@ -1577,8 +1667,27 @@ def qk_norm_store(q, k, v, heads, kv_heads, dim, vdim, q_weight, k_weight, eps, 
         qp, ldq, kp, ldk, vp, ldv, _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(out), _ptr(k_pool), _ptr(v_pool),
         _ptr(block_table), block_table.shape[1], _ptr(seq_of_token), _ptr(positions), page_size, n, heads, kv_heads, dim, vdim,
         int(bool(write)), _code(k_pool), _ptr(cos), _ptr(sin), rot, int(bool(interleaved)), _code(q), _ptr(q_bias), _ptr(k_bias),
-        _ptr(v_bias), int(unit_eps is not None), _stream()), "qk_norm_store")
+        _ptr(v_bias), int(unit_eps is not None), float(coef), int(every), _stream()), "qk_norm_store")
     return out
+
+
+@_flushes
+def pool_blocks(k_pool, v_pool, k_blocks, v_blocks, token_table, block_table, seq_of_token, positions, page_size,
+                block_page_size, block):
+    """The means of the keys and values of every block that a token of this step completes, into the blocks' pages."""
+    _, g, _, d = k_pool.shape
+    v = v_pool.shape[3]
+    entries = -(-block_page_size // block)
+    if len({t.dtype for t in (k_pool, v_pool, k_blocks, v_blocks)}) != 1:
+        raise TypeError("pool_blocks: tokens and blocks are kept in one dtype")
+    if k_blocks.shape[1:] != (g, entries, d) or v_blocks.shape[1:] != (g, entries, v):
+        raise ValueError("pool_blocks: the blocks' pages are [pages, kv_heads, ceil(page / block), size]")
+    for t in (k_pool, v_pool, k_blocks, v_blocks, token_table, block_table):
+        _dense(t, "pages and tables")
+    _check(_fn("attention_general", "akas_pool_blocks")(
+        _ptr(k_pool), _ptr(v_pool), _ptr(k_blocks), _ptr(v_blocks), _ptr(token_table), token_table.shape[1], _ptr(block_table),
+        block_table.shape[1], _ptr(seq_of_token), _ptr(positions), page_size, block_page_size, block, seq_of_token.numel(), g, d, v,
+        _code(k_pool), _stream()), "pool_blocks")
 
 
 # Which kernel runs the general attention over prompt portions in bfloat16: "mma" (default), the tensor-core kernel
@@ -1595,8 +1704,9 @@ general_splits = os.environ.get("AKAS_B200_GENERAL_SPLITS", "1") != "0"  # 0: a 
 @_flushes
 def attention_general(q, k_pool, v_pool, block_table, seq_of_token, positions, scale, window, keep_first, softcap,
                       r1, r2, sink, gate, page_size, ctx=None, sinks=None, out=None, out_scale=1.0, values_in_keys=0,
-                      gate_channels=False):
-    """``values_in_keys`` = V > 0: a key's row holds its value too, as its first V channels; ``v_pool`` is not read.
+                      gate_channels=False, blocks=None):
+    """``blocks`` = (k_blocks, v_blocks, block_table, page_size, block): what a token sees in front of its window (the
+    ``pool_blocks`` of its request). ``values_in_keys`` = V > 0: a key's row holds its value too, as its first V channels; ``v_pool`` is not read.
     ``gate_channels``: the gate has one logit per channel of a token's output row [N, heads * value_dim], not one per head."""
     n = q.shape[0]
     kh, d = k_pool.shape[1], k_pool.shape[3]
@@ -1622,6 +1732,23 @@ def attention_general(q, k_pool, v_pool, block_table, seq_of_token, positions, s
     elif out.shape != (n, heads * vd) or out.dtype != q.dtype:
         raise ValueError("attention_general: out must be [N, heads * value_dim] in q's dtype")
     op, ldo = _rows(out, "out")
+    if (r1 is None) != (r2 is None) and r1 is None:
+        raise ValueError("attention_general: a linear distance penalty is r1 alone")
+    kb = vb = None
+    block_tables, block_page, block = None, 0, 0
+    if blocks is not None:
+        kb, vb, block_tables, block_page, block = blocks
+        if kb.dtype != q.dtype or vb.dtype != q.dtype or kb.shape[1] != kh or kb.shape[3] != d or vb.shape[3] != vd:
+            raise ValueError("attention_general: blocks have the keys' and values' heads, sizes and dtype")
+        if not window or keep_first or r1 is not None or values_in_keys:
+            raise ValueError("attention_general: blocks lie in front of a window, without kept first tokens or a distance penalty")
+        _dense(kb, "k_blocks"), _dense(vb, "v_blocks"), _dense(block_tables, "the blocks' table")
+
+    def blocks_from(request):  # the blocks' arguments of a launch that starts at that request
+        if blocks is None:
+            return None, None, None, 0, 0, 0
+        return _ptr(kb), _ptr(vb), _ptr(block_tables[request:]), block_tables.shape[1], block_page, block
+
     tail = (_ptr(sinks), float(out_scale), ldo)
     options = (float(scale), int(window or 0), int(keep_first or 0), float(softcap or 0.0), _ptr(r1), _ptr(r2),
                int(bool(sink)), gp, ldg, page_size)
@@ -1647,13 +1774,14 @@ def attention_general(q, k_pool, v_pool, block_table, seq_of_token, positions, s
                 err = _fn("attention_general_tc", "akas_attention_general_tc")(
                     _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table[start:]), block_table.shape[1],
                     _ptr(ctx.cu_seqlens[start:]), _ptr(positions), op, *options, tiles, heads, kh, d, vd, requests,
-                    packed, *tail, _ptr(partial), splits, vpitch, channels, gate_code, _stream())
+                    packed, *tail, _ptr(partial), splits, vpitch, channels, gate_code, *blocks_from(start), _stream())
                 _check(err, "attention_general (tensor cores)")
             singles = 0
     if singles:
         _check(_fn("attention_general", "akas_attention_general")(
             _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), block_table.shape[1], _ptr(seq_of_token), _ptr(positions),
-            op, *options, singles, heads, kh, d, vd, _code(q), *tail, vpitch, channels, gate_code, _stream()), "attention_general")
+            op, *options, singles, heads, kh, d, vd, _code(q), *tail, vpitch, channels, gate_code, *blocks_from(0), _stream()),
+            "attention_general")
     return out
 
 
@@ -1776,7 +1904,8 @@ def head_linear(x, w, heads, gate=None, cos=None, sin=None, interleaved=False):
 
 
 @_flushes
-def moe_route(h, w_router, correction, groups, keep, top, scoring="softmax", renormalize=True, extra=0):
+def moe_route(h, w_router, correction, groups, keep, top, scoring="softmax", renormalize=True, extra=0, group_best=1,
+              weight_scale=1.0):
     """``extra`` = X > 0: the matrix has X more rows behind the R that compete; the sigmoids of their logits come back
     as a third result, float32 [N, X]."""
     n, c = h.shape
@@ -1792,8 +1921,8 @@ def moe_route(h, w_router, correction, groups, keep, top, scoring="softmax", ren
     extras = torch.empty((n, int(extra)), dtype=torch.float32, device=h.device) if extra else None
     _check(_fn("moe", "akas_moe_route")(hp, ldh, _ptr(_dense(w_router, "w_router")), _ptr(correction), _ptr(chosen),
                                        _ptr(weights), n, c, r, int(groups), int(keep), int(top), _code(h),
-                                       int(scoring == "sigmoid"), int(bool(renormalize)), int(extra), _ptr(extras), _stream()),
-           "moe_route")
+                                       int(scoring == "sigmoid"), int(bool(renormalize)), int(extra), _ptr(extras), int(group_best),
+                                       float(weight_scale), _stream()), "moe_route")
     return (chosen, weights, extras) if extra else (chosen, weights)
 
 
@@ -1815,7 +1944,7 @@ def _update_args(update, n, c):
     if update is None:
         return None, None, None, None, 0.0
     x, a, scale_a, scale_b, mult = update
-    for t in (x, a):
+    for t in (x, a) if a is not None else (x,):
         if t.dtype != torch.float32 or t.shape != (n, c) or not t.is_contiguous():
             raise ValueError("a residual update takes dense float32 tensors [N, C]")
     return _ptr(x), _ptr(a), _ptr(scale_a), _ptr(scale_b), float(mult)
@@ -1870,7 +1999,7 @@ def moe_experts(h, w_gate_up, w_down, chosen, weights, update=None, weight_input
     result. ``shared`` = (y float32 [N, C], gate float32 [N, 1] or None): y times its gate is added to the sum.
     The weighted sum of the chosen experts' results, float32 [N, C]. With ``update`` = (x, a, scale_a, scale_b, mult)
     the sum is not returned but added into the residual stream by the last kernel: x += mult * (scale_a * a + scale_b *
-    sum), in place; returns x. ``activation`` ("relu2", "gelu_tanh", "silu"; None: gated experts): experts without a gate,
+    sum) (``a`` None: none), in place; returns x. ``activation`` ("relu2", "gelu_tanh", "silu"; None: gated experts): experts without a gate,
     w_gate_up = w_up [E, F, C]."""
     n, c = h.shape
     experts, f2, _ = w_gate_up.shape

@@ -26,6 +26,46 @@ def embedding(token_ids, table):
     return table[token_ids.long()].to(torch.float32)
 
 
+def bigram_embedding(token_ids, table, pairs, mul_prev, mul_cur, state, cu_seqlens, seq_of_token, slots, out=None):
+    """table[token] plus a row of ``pairs`` [buckets + 1, C], float32 [N, C]: row (previous * mul_prev + token * mul_cur)
+    mod buckets with the token in front of it in its request, row ``buckets`` for a request's first token. ``state``
+    int32 [slots, 1] holds the last token of the steps before plus one (0: none yet) and receives this step's. Tokens of
+    no request get their row of ``table`` alone. ``out`` [2, N, C]: the result is written to both halves, and the second
+    is returned."""
+    buckets = pairs.shape[0] - 1
+    value = table[token_ids.long()].to(torch.float32)
+    ids, cu, seqs = token_ids.tolist(), cu_seqlens.tolist(), seq_of_token.tolist()
+    slot_of = slots.tolist()
+    held = {r: int(state[slot, 0]) for r, slot in enumerate(slot_of) if slot >= 0}
+    for n, (token, r) in enumerate(zip(ids, seqs)):
+        if r < 0:
+            continue
+        previous = ids[n - 1] if n > cu[r] else held[r] - 1
+        row = buckets if previous < 0 else (previous * mul_prev + token * mul_cur) % buckets
+        value[n] += pairs[row].to(torch.float32)
+    for r, slot in enumerate(slot_of):
+        if slot >= 0 and cu[r + 1] > cu[r]:
+            state[slot, 0] = ids[cu[r + 1] - 1] + 1
+    if out is not None:
+        out[:2] = value
+        return out[1]
+    return value
+
+
+def depth_average(history, count, weights, out, rows=None, norm=None):
+    """sum_j weights[j] * history[j] over j < count, float32 [N, C] (or of the rows ``rows`` alone, [M, C]), for float32
+    history [.., N, C]; written to ``out`` where that is given. ``norm`` = (weight, eps, zero_centered, dtype): also that
+    RMSNorm of the result. Returns (result, normed result or None)."""
+    picked = history[:count] if rows is None else history[:count][:, rows.long()]
+    value = torch.einsum("jnc,j->nc", picked, weights.to(torch.float32))
+    if out is not None:
+        value = out.copy_(value)
+    if norm is None:
+        return value, None
+    weight, eps, zero_centered, dtype = norm
+    return value, rmsnorm(value, weight, eps, zero_centered, dtype)
+
+
 def rmsnorm(x, weight, eps, zero_centered, out_dtype, rows=None):
     if rows is not None:
         x = x[rows.long()]
@@ -341,6 +381,26 @@ def decay_scan(q, k, v, decay, state, cu_seqlens, slots, heads, dim, vdim, q_sca
     return o.reshape(n, heads * vdim)
 
 
+def hgrn2_scan(q, f, v, f_bias, lower, state, cu_seqlens, slots, heads, dim, vdim, write=True, longest=None):
+    """Per request and head, token by token: S <- diag(g_t) S + (1 - g_t) v_t^T; o_t = S^T silu(q_t), with the gate
+    g = lower + (1 - lower) sigmoid(f + f_bias) per key channel (f_bias, lower float32 [heads * dim]).
+    q, f [N, heads * dim], v [N, heads * vdim] -> o float32 [N, heads * vdim]; state [slots, heads, vdim, dim]."""
+    n = q.shape[0]
+    o = torch.zeros((n, heads, vdim), dtype=torch.float32, device=q.device)
+    qf, vf = q.to(torch.float64), v.to(torch.float64).reshape(n, heads, vdim)
+    qf = (qf * torch.sigmoid(qf)).reshape(n, heads, dim)
+    low = lower.to(torch.float64)
+    g = (low + (1.0 - low) * torch.sigmoid(f.to(torch.float64) + f_bias.to(torch.float64))).reshape(n, heads, dim)
+    for slot, a, b in _requests(cu_seqlens, slots):
+        s = state[slot].to(torch.float64)
+        for t in range(a, b):
+            s = g[t][:, None, :] * s + vf[t][:, :, None] * (1.0 - g[t])[:, None, :]
+            o[t] = torch.einsum("hvd,hd->hv", s, qf[t]).to(torch.float32)
+        if write:
+            state[slot] = s.to(torch.float32)
+    return o.reshape(n, heads * vdim)
+
+
 def causal_conv_silu(x, taps, state, cu_seqlens, seq_of_token, slots, write=True):
     """silu of a causal depthwise convolution over each request's tokens: y_t = silu(sum_j taps[:, j] x_(t - L + 1 + j)),
     inputs before the step's first token from ``state`` (zero at a request's start). x [N, C] -> float32 [N, C]."""
@@ -397,7 +457,7 @@ def delta_scan(q, k, v, beta, g, state, cu_seqlens, slots, heads, kv_heads, dim,
 
 def gated_rmsnorm(o, weight, eps, gate, heads, vdim, out_dtype, gate_activation="silu", out=None, out_scale=1.0):
     """Each head of o [N, heads * vdim] over its root mean square (eps under the root), times weight [vdim] (None: ones), times
-    silu(gate) [N, heads * vdim] (or, ``gate_activation="sigmoid"``, sigmoid(gate)), times ``out_scale``; written into
+    silu(gate) [N, heads * vdim] (or, ``gate_activation="sigmoid"``, sigmoid(gate); ``gate`` None: no gate), times ``out_scale``; written into
     ``out`` (a view [N, heads * vdim] whose rows may be parts of wider rows) where that is given. A norm over all
     heads together is the call with heads = 1."""
     n = o.shape[0]
@@ -405,8 +465,10 @@ def gated_rmsnorm(o, weight, eps, gate, heads, vdim, out_dtype, gate_activation=
     of = of / torch.sqrt((of * of).mean(dim=-1, keepdim=True) + eps)
     if weight is not None:
         of = of * weight.to(torch.float64)
-    gf = gate.to(torch.float64)
-    act = torch.sigmoid(gf) if gate_activation == "sigmoid" else gf * torch.sigmoid(gf)
+    act = 1.0
+    if gate is not None:
+        gf = gate.to(torch.float64)
+        act = torch.sigmoid(gf) if gate_activation == "sigmoid" else gf * torch.sigmoid(gf)
     y = of.reshape(n, heads * vdim) * act * out_scale
     if out is not None:
         out.copy_(y.to(out.dtype))
@@ -419,13 +481,14 @@ def gated_rmsnorm(o, weight, eps, gate, heads, vdim, out_dtype, gate_activation=
 
 def qk_norm_store(q, k, v, heads, kv_heads, dim, vdim, q_weight, k_weight, eps, k_pool, v_pool, block_table,
                   seq_of_token, positions, page_size, write=True, cos=None, sin=None, interleaved=False,
-                  q_bias=None, k_bias=None, v_bias=None, unit_eps=None):
+                  q_bias=None, k_bias=None, v_bias=None, unit_eps=None, temperature=None):
     """First, where biases (float32 [heads * dim], [kv_heads * dim], [kv_heads * vdim]) are given, q, k and v plus
     their biases (q, k and v may then be float32 results of a product, rounded here for the first time). Then
     per-head RMSNorm (plain weight; None: no norm) of q [N, heads * dim] and k [N, kv_heads * dim], then, where
     ``cos`` and ``sin`` (float32 [N, rot / 2]) are given, the rotation of the first ``rot`` channels of every head of
     q and k: channel 2i with 2i + 1 (``interleaved``) or i with i + rot / 2. Then, where ``unit_eps`` is given, every
-    head of q and k over sqrt(mean of its dim squares + unit_eps), without a weight. k and the untouched v [N, kv_heads * vdim]
+    head of q and k over sqrt(mean of its dim squares + unit_eps), without a weight. ``temperature`` = (coef, every): q is
+    then multiplied by 1 + coef * ln(floor((position + 1) / every) + 1). k and the untouched v [N, kv_heads * vdim]
     go into the pages (k pages [.., kv_heads, page, dim], v pages [.., kv_heads, page, vdim]); returns q, contiguous,
     in the pools' dtype."""
     n = q.shape[0]
@@ -463,6 +526,10 @@ def qk_norm_store(q, k, v, heads, kv_heads, dim, vdim, q_weight, k_weight, eps, 
         qf, kf = turn(qf), turn(kf)
     if unit_eps is not None:
         qf, kf = (x * torch.rsqrt((x * x).mean(dim=-1, keepdim=True) + unit_eps) for x in (qf, kf))
+    if temperature is not None:
+        coef, every = temperature
+        stretches = torch.div(positions.long() + 1, every, rounding_mode="floor").to(torch.float64)
+        qf = qf * (1.0 + coef * torch.log(stretches + 1.0)).to(torch.float32)[:, None, None]
     if write:
         live, page, off = _page_addresses(block_table, seq_of_token, positions, page_size)
         k_pool[page[live], :, off[live]] = kf[live].to(k_pool.dtype)
@@ -470,14 +537,39 @@ def qk_norm_store(q, k, v, heads, kv_heads, dim, vdim, q_weight, k_weight, eps, 
     return qf.reshape(n, heads * dim).to(k_pool.dtype).contiguous()
 
 
+def _block_entry(block_table, r, b, page_size, block):
+    """(page, entry) of block number(s) ``b`` of request ``r``: the page of the block's last token, and the block's place
+    among those that end in that page."""
+    last = b * block + block - 1
+    page = last // page_size
+    return block_table[r, page].long(), b - page * page_size // block
+
+
+def pool_blocks(k_pool, v_pool, k_blocks, v_blocks, token_table, block_table, seq_of_token, positions, page_size,
+                block_page_size, block):
+    """For every token of the step that is the last of its block of ``block`` tokens: the means of the block's keys and
+    values as their pages hold them (summed in float32) go to the block's entry of ``k_blocks`` and ``v_blocks`` [pages,
+    kv_heads, ceil(block_page_size / block), size]."""
+    for r, p in zip(seq_of_token.tolist(), positions.tolist()):
+        if r < 0 or (p + 1) % block:
+            continue
+        idx = torch.arange(p - block + 1, p + 1, device=k_pool.device)
+        pages, offs = token_table[r, idx // page_size].long(), idx % page_size
+        page, entry = _block_entry(block_table, r, torch.tensor(p // block), block_page_size, block)
+        for pool, blocks in ((k_pool, k_blocks), (v_pool, v_blocks)):
+            blocks[page, :, entry] = pool[pages, :, offs].to(torch.float32).mean(dim=0).to(blocks.dtype)
+
+
 def attention_general(q, k_pool, v_pool, block_table, seq_of_token, positions, scale, window, keep_first, softcap,
                       r1, r2, sink, gate, page_size, ctx=None, sinks=None, out=None, out_scale=1.0, values_in_keys=0,
-                      gate_channels=False):
-    """``values_in_keys`` = V > 0: a key's row holds its value too, as its first V channels (``v_pool`` is not read).
+                      gate_channels=False, blocks=None):
+    """``blocks`` = (k_blocks, v_blocks, table, page_size, block), with a window: a token at position i also sees every
+    block b of ``block`` tokens with (b + 1) * block - 1 <= i - window, as one key and one value (see ``pool_blocks``), in
+    the same softmax. ``values_in_keys`` = V > 0: a key's row holds its value too, as its first V channels (``v_pool`` is not read).
     ``gate_channels``: ``gate`` is [N, heads * vdim], one logit per channel of the output, not one per head.
     Attention of every token over the keys of its request that it sees: j <= i and (no window, or i - j < window,
     or j < keep_first). score = q . k * scale; with softcap, cap * tanh(score / cap); with r1 and r2 (float32
-    [heads]), minus r1_h * ln(1 + r2_h * (i - j)); softmax over the keys, with ``sink`` one more term exp(0) in the
+    [heads]), minus r1_h * ln(1 + r2_h * (i - j)), with r1 alone minus r1_h * (i - j); softmax over the keys, with ``sink`` one more term exp(0) in the
     denominator, or with ``sinks`` (float32 [heads]) the term exp(sinks_h); the head's output times
     sigmoid(gate[n, h]) where ``gate`` [N, heads] is given, times ``out_scale``.
     q [N, heads * dim] -> [N, heads * vdim] in q's dtype, written into ``out`` (rows may be parts of wider rows) where given."""
@@ -501,12 +593,21 @@ def attention_general(q, k_pool, v_pool, block_table, seq_of_token, positions, s
         offs = idx % page_size
         keys = k_pool[pages, :, offs].to(torch.float64)  # [S, kh, d]
         vals = v_pool[pages, :, offs].to(torch.float64)
+        if blocks is not None:
+            k_blocks, v_blocks, table, block_page, block = blocks
+            b = torch.arange(max(0, p - window + 1) // block, device=q.device)
+            page, entry = _block_entry(table, r, b, block_page, block)
+            keys = torch.cat([keys, k_blocks[page, :, entry].to(torch.float64)])
+            vals = torch.cat([vals, v_blocks[page, :, entry].to(torch.float64)])
         qt = q[t].reshape(kh, group, d).to(torch.float64)
         s = torch.einsum("kgd,skd->kgs", qt, keys) * scale
         if softcap:
             s = softcap * torch.tanh(s / softcap)
         if r1 is not None:
             dist = (p - idx).to(torch.float64)
+            if r2 is None:
+                s = s - r1.to(torch.float64).reshape(kh, group, 1) * dist
+        if r1 is not None and r2 is not None:
             s = s - r1.to(torch.float64).reshape(kh, group, 1) * torch.log1p(r2.to(torch.float64).reshape(kh, group, 1) * dist)
         top = s.max(dim=-1, keepdim=True).values
         level = None
@@ -640,7 +741,8 @@ def head_linear(x, w, heads, gate=None, cos=None, sin=None, interleaved=False):
 # --------------------------------------------------------------------------- routed experts, parallel blocks
 
 
-def moe_route(h, w_router, correction, groups, keep, top, scoring="softmax", renormalize=True, extra=0):
+def moe_route(h, w_router, correction, groups, keep, top, scoring="softmax", renormalize=True, extra=0, group_best=1,
+              weight_scale=1.0):
     """For every row of h [N, C]: scores = softmax(h . w_router^T) over the R router outputs (float32 w_router
     [R, C]); choice scores = scores + correction [R]; the outputs form ``groups`` equal groups of neighbours whose
     score is their largest choice score, and only outputs of the ``keep`` best groups can be chosen; the ``top``
@@ -648,7 +750,8 @@ def moe_route(h, w_router, correction, groups, keep, top, scoring="softmax", ren
     chosen outputs in the order of their choice scores and their plain scores over their sum (+ 1e-20).
     Without a correction the choice goes by the logits, which order as the scores do. ``scoring="sigmoid"``: a score is
     the sigmoid of its logit; ``correction`` None: none; ``renormalize`` False: the
-    weights are the chosen scores as they are. ``extra`` = X > 0: w_router has X more rows [R + X, C] that take no part
+    weights are the chosen scores as they are; ``group_best`` B: a group's score is the sum of its B largest choice
+    scores; ``weight_scale``: the weights times this constant. ``extra`` = X > 0: w_router has X more rows [R + X, C] that take no part
     in the choice; the sigmoids of their logits are returned as a third result, float32 [N, X]."""
     n = h.shape[0]
     r = w_router.shape[0] - extra
@@ -656,10 +759,12 @@ def moe_route(h, w_router, correction, groups, keep, top, scoring="softmax", ren
     s = torch.softmax(z[:, :r], dim=-1) if scoring == "softmax" else torch.sigmoid(z[:, :r])
     if correction is not None:
         pick = s + correction.to(torch.float32)
+    elif group_best > 1:  # (sums of logits would not order as sums of scores do)
+        pick = s.clone()
     else:  # the logits order as their scores do, and still compare where two scores round to one
         pick = z[:, :r].clone()
     if groups > 1 and keep < groups:
-        best = pick.reshape(n, groups, r // groups).max(dim=-1).values
+        best = pick.reshape(n, groups, r // groups).topk(min(group_best, r // groups), dim=-1).values.sum(dim=-1)
         order = torch.argsort(best, dim=-1, descending=True, stable=True)
         stays = torch.zeros((n, groups), dtype=torch.bool, device=h.device)
         stays.scatter_(1, order[:, :keep], True)
@@ -668,6 +773,8 @@ def moe_route(h, w_router, correction, groups, keep, top, scoring="softmax", ren
     w = torch.gather(s, 1, chosen)
     if renormalize:
         w = w / (w.sum(dim=-1, keepdim=True) + 1e-20)
+    if weight_scale != 1.0:
+        w = w * weight_scale
     if extra:
         return chosen.to(torch.int32), w, torch.sigmoid(z[:, r:]).contiguous()
     return chosen.to(torch.int32), w
@@ -677,7 +784,7 @@ def moe_experts(h, w_gate_up, w_down, chosen, weights, update=None, weight_input
     """``activation`` (None: gated experts as below): experts without a gate, w_down[e] act(w_up[e] h) with w_gate_up =
     w_up [E, F, C] and act "relu2", "gelu_tanh" or "silu". ``weight_input``: the weight multiplies the expert's input, out[n] = sum_k expert(weights[n, k] h[n]) (computed
     as silu(w g) * (w u) on the float32 sums g, u of the unweighted row). ``shared`` = (y float32 [N, C], gate float32
-    [N, 1] or None): y, times its gate, is added to the sum. With ``update`` = (x, a, scale_a, scale_b, mult): x += mult * (scale_a * a + scale_b * out) in place, returns x. Else
+    [N, 1] or None): y, times its gate, is added to the sum. With ``update`` = (x, a, scale_a, scale_b, mult): x += mult * (scale_a * a + scale_b * out) in place (``a`` None: x += mult * scale_b * out), returns x. Else
     out[n] = sum_k weights[n, k] * expert_(chosen[n, k])(h[n]) in float32 [N, C]. Expert e < E computes
     w_down[e] (silu(gate) * up) with [gate; up] = w_gate_up[e] h (w_gate_up [E, 2 F, C], w_down [E, C, F]; the hidden
     activations are rounded to h's dtype, as the kernels round them); an expert number from E on returns h itself."""
@@ -706,6 +813,8 @@ def moe_experts(h, w_gate_up, w_down, chosen, weights, update=None, weight_input
         out += y if gate is None else gate.reshape(n, 1) * y
     if update is not None:
         x, a, scale_a, scale_b, mult = update
+        if a is None:
+            return scaled_add(x, out, scale_b, None, None, mult)
         return scaled_add(x, a, scale_a, out, scale_b, mult)
     return out
 

@@ -4,6 +4,7 @@ from .base import (
     FeedForward,
     Mixer,
     Normed,
+    PagedBlocksSpec,
     PagedKVSpec,
     PagedLatentSpec,
     PagedSpec,
@@ -28,13 +29,13 @@ from .moe import RoutedExperts
 from .norm import DynamicTanh, RMSNorm
 from .parallel import ParallelMixer
 from .polynorm import PolyNormMLP
-from .recurrent import DecayedLinearAttention, GatedDelta, GatedLinearAttention
+from .recurrent import HGRN2, DecayedLinearAttention, GatedDelta, GatedLinearAttention
 from .rope import Rope
 from .shortconv import ShortConv
 from .swiglu import SwiGLU
 
 __all__ = [
-    "ARRANGEMENTS", "MLP", "Attention", "Block", "DynamicTanh", "GatedMLP", "LatentAttention", "PagedLatentSpec", "DecayedLinearAttention", "ParallelMixer", "RoutedExperts", "FeedForward", "GatedDelta", "GatedLinearAttention", "Mixer", "PolyNormMLP", "Normed", "PagedKVSpec", "PagedSpec", "Param", "Part", "RMSNorm",
+    "ARRANGEMENTS", "MLP", "Attention", "Block", "DynamicTanh", "GatedMLP", "LatentAttention", "PagedLatentSpec", "DecayedLinearAttention", "ParallelMixer", "RoutedExperts", "FeedForward", "HGRN2", "PagedBlocksSpec", "GatedDelta", "GatedLinearAttention", "Mixer", "PolyNormMLP", "Normed", "PagedKVSpec", "PagedSpec", "Param", "Part", "RMSNorm",
     "Rope", "Runtime", "ShortConv", "StateSpec", "SwiGLU", "build_part", "project", "project_swiglu", "register_ffn", "register_mixer",
     "register_norm", "register_position",
 ]

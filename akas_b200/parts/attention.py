@@ -12,10 +12,14 @@ and to itself; the output product, added to the residual.
 A layer whose spec asks for more than that (value heads of another size than the keys', a capped score, a
 logarithmic distance penalty, first tokens kept behind the window, a sink in the softmax's denominator (exp(0) or a
 learned logit per head), a gate per head on the output, values that are the keys as projected, rotary pairs of
-neighbouring channels, biases on q, k and v, no keys and values of its own but another layer's cache) runs the same
+neighbouring channels, biases on q, k and v, no keys and values of its own but another layer's cache, queries times a
+temperature that grows with the position, a linear distance penalty, whole blocks of tokens seen as their means in
+front of a window) runs the same
 steps on the general kernels: one product for q, k, v and the gate's
 logits, QK-norm, rotation and page write (``ops.qk_norm_store``), attention with the options as arguments
-(``ops.attention_general``), the output product. ``core`` is that sequence without the two products, for a mixer
+(``ops.attention_general``), the output product. A layer that sees blocks keeps two caches, the tokens' pages (given
+back behind the window) and the blocks' (``PagedBlocksSpec``, kept for ever); a block's means are made from the cached
+rows of its tokens in the step that brings its last token, before the attention (``ops.pool_blocks``). ``core`` is that sequence without the two products, for a mixer
 that stacks this one's matrices with its neighbours' (``parts/parallel.py``).
 """
 
@@ -23,7 +27,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import Mixer, PagedKVSpec, Param, build_part, project, register_mixer, renamed, stack_rows
+from .base import Mixer, PagedBlocksSpec, PagedKVSpec, Param, build_part, project, register_mixer, renamed, stack_rows
 
 
 class Attention(Mixer):
@@ -44,6 +48,7 @@ class Attention(Mixer):
         if s.num_heads % s.num_kv_heads:
             raise ValueError(f"{s.num_heads} heads are not a multiple of {s.num_kv_heads} key/value heads")
         self.general = bool(getattr(s, "general", False))
+        self.takes_residual_scale = self.general
         if not self.general and (s.head_dim % 16 or s.head_dim > 256):
             raise ValueError(f"head_dim {s.head_dim} must be a multiple of 16, at most 256")
         if s.sink not in (False, True, "learned"):
@@ -57,6 +62,12 @@ class Attention(Mixer):
         self.unit_eps = getattr(s, "qk_unit_eps", None)
         if self.unit_eps is not None and s.qk_norm is not None:
             raise ValueError("q and k are normed in front of the position encoding (qk_norm) or behind it (qk_unit_eps), not both")
+        self.pool = getattr(s, "pool", None) or 0
+        if self.pool and (not s.window or s.keep_first or s.distance_bias):
+            raise ValueError("blocks of tokens need a window, and take neither kept first tokens nor a distance penalty")
+        if self.general and s.distance_bias not in (False, True, "linear"):
+            raise ValueError(f"unknown distance bias {s.distance_bias!r}; known: False, True, 'linear'")
+        self.out_biased = bool(getattr(s, "out_bias", False))
         self.own_kv = bool(getattr(s, "own_kv", True))
         self.biased = bool(getattr(s, "bias", False))
         if not self.own_kv and getattr(s, "values_are_keys", False):
@@ -71,7 +82,7 @@ class Attention(Mixer):
             raise ValueError("heads are normed behind a position encoding by rotary tables only")
         self.w_qkv = None
         self.w_out = None
-        self.r1 = self.r2 = self.sinks = self.bias = None
+        self.r1 = self.r2 = self.sinks = self.bias = self.b_out = None
 
     def _n(self, local):
         return renamed(self.spec, local)
@@ -99,11 +110,13 @@ class Attention(Mixer):
             for local in ("q_proj.weight", "k_proj.weight", "v_proj.weight"):
                 if self._n(local) in p:
                     p[self._n(local) + ".b"] = Param((p[self._n(local)].shape[0],), role="vector")
+        if self.out_biased:
+            p[self._n("out_proj.weight") + ".b"] = Param((s.hidden_size,), role="vector")
         if self.general and s.sink == "learned":
             p[self._n("sink")] = Param((s.num_heads,), role="vector")
         if self.general and s.gate is not None:
             p[self._n("gate.weight")] = Param((self._gate_rows(), s.hidden_size))
-        if self.general and s.distance_bias:
+        if self.general and s.distance_bias is True:
             p[self._n("r1")] = Param((s.num_heads,), role="vector")
             p[self._n("r2")] = Param((s.num_heads,), role="vector", mean=0.5)
         if self.q_norm is not None:
@@ -127,13 +140,20 @@ class Attention(Mixer):
                 self.bias = torch.cat([get(name + ".b") for name in names]).contiguous()
             if self.spec.sink == "learned":
                 self.sinks = get(self._n("sink"))
-            if self.spec.distance_bias:
+            if self.spec.distance_bias is True:
                 self.r1, self.r2 = get(self._n("r1")), get(self._n("r2"))
         else:
             self.w_qkv = torch.cat(
                 [get(self._n("q_proj.weight")), get(self._n("k_proj.weight")), get(self._n("v_proj.weight"))], dim=0
             ).contiguous()
         self.w_out = get(self._n("out_proj.weight"))
+        if self.out_biased:  # what is added beside a residual: the constant that multiplies the result multiplies it too
+            b = get(self._n("out_proj.weight") + ".b")
+            self.b_out = b if self.residual_scale == 1.0 else (b * self.residual_scale).contiguous()
+        if self.general and self.spec.distance_bias == "linear":
+            h = self.spec.num_heads
+            self.r1 = torch.tensor([2.0 ** (-8.0 * (a + 1) / h) for a in range(h)], dtype=torch.float64).to(
+                device=self.w_out.device, dtype=torch.float32)
         if self.q_norm is not None:
             self.q_norm.weight = get(self._n("q_norm.weight"))
             self.k_norm.weight = get(self._n("k_norm.weight"))
@@ -143,8 +163,11 @@ class Attention(Mixer):
         if not self.own_kv:
             raise ValueError("this attention layer keeps no keys and values: the run order must give it another layer's cache")
         if self.general:
-            return PagedKVSpec(s.num_kv_heads, s.head_dim, s.window, keep_first=s.keep_first if s.window else 0,
-                               v_head_dim=s.value_dim)
+            tokens = PagedKVSpec(s.num_kv_heads, s.head_dim, s.window, keep_first=s.keep_first if s.window else 0,
+                                 v_head_dim=s.value_dim, pool=self.pool)
+            if not self.pool:
+                return tokens
+            return tokens, PagedBlocksSpec(self.pool, s.num_kv_heads, s.head_dim, s.value_dim)
         return PagedKVSpec(s.num_kv_heads, s.head_dim, s.window)
 
     @property
@@ -161,6 +184,7 @@ class Attention(Mixer):
         s, ops = self.spec, self.rt.ops
         if not self.own_kv and write:
             raise ValueError("a layer without keys and values of its own writes no cache")
+        cache, blocks = cache if self.pool else (cache, None)
         nq = s.num_heads * s.head_dim
         nk = s.num_kv_heads * s.head_dim if self.own_kv else 0
         nv = 0 if s.values_are_keys or not self.own_kv else s.num_kv_heads * s.value_dim
@@ -179,12 +203,20 @@ class Attention(Mixer):
         if self.bias is not None:
             rotary.update(q_bias=self.bias[:nq], k_bias=self.bias[nq : nq + nk] if nk else None,
                           v_bias=self.bias[nq + nk : nq + nk + nv] if nv else None)
+        if s.q_temperature is not None:
+            rotary.update(temperature=s.q_temperature)
         qn = ops.qk_norm_store(
             q, k, v, s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim,
             self.q_norm.weight if norm else None, self.k_norm.weight if norm else None, norm.eps if norm else 0.0,
             cache.k, cache.v, table, ctx.seq_of_token, ctx.positions, cache.page_size, write=write, **rotary,
         )
         more = {}
+        if blocks is not None:
+            block_table = ctx.block_table(blocks.group)
+            if write:
+                ops.pool_blocks(cache.k, cache.v, blocks.k, blocks.v, table, block_table, ctx.seq_of_token, ctx.positions,
+                                cache.page_size, blocks.page_size, self.pool)
+            more["blocks"] = (blocks.k, blocks.v, block_table, blocks.page_size, self.pool)
         if self.sinks is not None:
             more["sinks"] = self.sinks
         if out is not None:
@@ -201,8 +233,14 @@ class Attention(Mixer):
     def _forward_general(self, x, ctx, cache, residual, write, out_dtype=None):
         # with biases the product leaves float32, so that product plus bias is rounded once (by the kernel that adds it)
         proj = project(self.rt, x, self.w_qkv, out_dtype=torch.float32 if self.bias is not None else None)
-        out = self.core(proj, ctx, cache, write)
-        return project(self.rt, out, self.w_out, out_dtype=out_dtype, residual=residual)
+        # a constant on what goes into the residual rides on the heads' outputs (and on the bias, which has it already)
+        out = self.core(proj, ctx, cache, write, out_scale=1.0 if residual is None else self.residual_scale)
+        return self._output(out, out_dtype, residual)
+
+    def _output(self, out, out_dtype, residual):
+        if residual is None and self.b_out is not None and self.residual_scale != 1.0:
+            raise ValueError("this layer's output bias was loaded for a scaled residual")
+        return project(self.rt, out, self.w_out, out_dtype=out_dtype, residual=residual, bias=self.b_out)
 
     def forward(self, x, ctx, cache=None, residual=None, write=True, out_dtype=None):
         s, ops = self.spec, self.rt.ops
@@ -227,7 +265,7 @@ class Attention(Mixer):
                 ctx, write=write, **unit,
             )
             if out is not None:
-                return project(self.rt, out, self.w_out, out_dtype=out_dtype, residual=residual)
+                return self._output(out, out_dtype, residual)
         store = write and fused
         q = ops.qk_norm_rope_store(
             qkv, s.num_heads, s.num_kv_heads, s.head_dim,
@@ -248,7 +286,7 @@ class Attention(Mixer):
             q, cache.k, cache.v, ctx.block_table(cache.group), ctx.seq_of_token, ctx.positions,
             self.scale, s.window, cache.page_size, ctx,
         )
-        return project(self.rt, out, self.w_out, out_dtype=out_dtype, residual=residual)
+        return self._output(out, out_dtype, residual)
 
 
 register_mixer("attention", Attention)

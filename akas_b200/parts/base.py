@@ -17,6 +17,9 @@ Interfaces (duck-typed; these base classes only document and give defaults):
   write)``.
 * FeedForward: ``params()``, ``load(get)``, ``forward(x, ctx, residual)``.
 
+A mixer or feed-forward that can multiply what it adds into a residual by a constant sets ``takes_residual_scale``; the
+block then sets its ``residual_scale``.
+
 ``forward`` of a mixer or feed-forward gets the normed activations ``x`` ``[N, C]``
 in the compute dtype and, when ``residual`` is given (float32 ``[N, C]``), returns
 ``residual + result`` in float32 (it may add in place; the fused kernels do).
@@ -74,12 +77,15 @@ class PagedSpec:
     page_size: Optional[int] = None
     dtype: Optional[torch.dtype] = None
     keep_first: int = 0  # with a window: the first keep_first tokens are read for ever, so their pages are never given back
+    # with a window: tokens are read once more when the block of ``pool`` tokens they are in is complete, so a page stays
+    # until the blocks it holds a part of are
+    pool: int = 0
 
     def pools(self, page_size: int) -> Dict[str, Tuple[int, ...]]:
         raise NotImplementedError
 
     def paging(self) -> tuple:
-        return (self.window, self.page_size, self.keep_first if self.window else 0)
+        return (self.window, self.page_size, self.keep_first if self.window else 0, self.pool if self.window else 0)
 
 
 @dataclass(frozen=True)
@@ -94,10 +100,30 @@ class PagedKVSpec(PagedSpec):
     dtype: Optional[torch.dtype] = None
     keep_first: int = 0
     v_head_dim: Optional[int] = None
+    pool: int = 0
 
     def pools(self, page_size: int) -> Dict[str, Tuple[int, ...]]:
         return {"k": (self.num_kv_heads, page_size, self.head_dim),
                 "v": (self.num_kv_heads, page_size, self.v_head_dim or self.head_dim)}
+
+
+@dataclass(frozen=True)
+class PagedBlocksSpec(PagedSpec):
+    """One key and one value for every whole block of ``block`` tokens, for ever: a block lies in the page of its last
+    token, so a page of ``page_size`` tokens holds at most ceil(page_size / block) of them, in their order:
+    ``[kv_heads, ceil(page_size / block), head_dim]`` (values: ``v_head_dim``). Block b of a request is entry
+    b - floor(first / block) of its page, with ``first`` the page's first position."""
+
+    block: int = 16
+    num_kv_heads: int = 1
+    head_dim: int = 16
+    v_head_dim: Optional[int] = None
+    page_size: Optional[int] = None
+    dtype: Optional[torch.dtype] = None
+
+    def pools(self, page_size: int) -> Dict[str, Tuple[int, ...]]:
+        entries = -(-page_size // self.block)
+        return {"k": (self.num_kv_heads, entries, self.head_dim), "v": (self.num_kv_heads, entries, self.v_head_dim or self.head_dim)}
 
 
 @dataclass(frozen=True)
@@ -235,6 +261,10 @@ class Part:
     # that defers launches (a decode step run as one chain) may keep deferring across it. A part that computes with
     # torch directly leaves this False, and the decoder makes everything pending run before the part does.
     chain_safe = False
+    # True: the part adds ``residual_scale`` times its result into a residual (a constant that the block sets before
+    # loading); a part that leaves this False is asked for its result and the block adds it.
+    takes_residual_scale = False
+    residual_scale = 1.0
 
     def __init__(self, spec, runtime: Runtime):
         self.spec = spec

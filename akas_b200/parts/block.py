@@ -1,7 +1,8 @@
 """A block: a mixer and (unless the layer has none) a feed-forward, each behind its norm, around a float32 residual stream.
 
 ``pre_norm`` (the only arrangement LFM2 uses, src/akas/models/lfm2/_composition.py:189,308-309,356
-in kreasof-ai/akas): h += mixer(norm(h)); h += ffn(norm(h)). ``parallel``: one norm n = norm(h) that the mixer and
+in kreasof-ai/akas): h += mixer(norm(h)); h += ffn(norm(h)), each result times a constant where the layer has one (by the
+part itself where it offers that, so that nothing is written by itself). ``parallel``: one norm n = norm(h) that the mixer and
 the feed-forward both read, or a norm for each, both of the same h; h += m * (s1 * mixer(n) + s2 * ffn(n)) with a
 constant m and a learned scale per channel for each sublayer (the two results are float32 and meet the residual stream
 in one kernel; without constant and scales, a feed-forward in two halves adds into the stream like the mixer does, both
@@ -18,18 +19,29 @@ import torch
 from .base import Param, Runtime, build_part, load_norm, norm_pair, norm_params
 
 
-def _normed(norm, part, h):
-    """The norm's output for ``part``: left to the part's first product when both sides can do that."""
+def _normed(norm, part, h, ready=None):
+    """The norm's output for ``part``: left to the part's first product when both sides can do that. ``ready``: the
+    output, if whoever made h has made it too."""
+    if ready is not None:
+        return ready
     if getattr(part, "takes_normed", False) and hasattr(norm, "lazy"):
         return norm.lazy(h)
     return norm.forward(h)
 
 
-def _pre_norm(block, h, ctx, cache, write):
-    h = block.mixer.forward(_normed(block.mixer_norm, block.mixer, h), ctx, cache, residual=h, write=write)
+def _pre_norm(block, h, ctx, cache, write, normed=None):
+    h = _add_result(block, block.mixer, h, _normed(block.mixer_norm, block.mixer, h, normed), ctx, cache, write=write)
     if block.ffn is None:
         return h
-    return block.ffn.forward(_normed(block.ffn_norm, block.ffn, h), ctx, residual=h)
+    return _add_result(block, block.ffn, h, _normed(block.ffn_norm, block.ffn, h), ctx)
+
+
+def _add_result(block, part, h, *args, **kwargs):
+    """h += residual_multiplier * part(...): by the part itself where it takes the constant."""
+    mult = block.spec.residual_multiplier
+    if getattr(part, "residual_scale", 1.0) == mult:
+        return part.forward(*args, residual=h, **kwargs)
+    return block.mixer.rt.ops.scaled_add(h, _float32_result(part, *args, residual=None, **kwargs), None, None, None, mult)
 
 
 def _float32_result(part, *args, **kwargs):
@@ -109,6 +121,12 @@ class Block:
         if spec.arrangement == "sandwich" and (self.mixer_post_norm is None or (self.ffn is not None and self.ffn_post_norm is None)):
             raise ValueError("the sandwich arrangement needs a norm behind each sublayer")
         self._run = ARRANGEMENTS[spec.arrangement]
+        # Whether ``forward`` takes the first norm's output from whoever made h (a kernel that makes h can make both)
+        self.takes_ready_norm = spec.arrangement == "pre_norm"
+        if spec.arrangement == "pre_norm":
+            for part in (self.mixer, self.ffn):
+                if getattr(part, "takes_residual_scale", False):
+                    part.residual_scale = spec.residual_multiplier
         self.mixer_scale = self.ffn_scale = None  # the parallel arrangement's scales per channel, where the layer names them
         # Whether every part of the block reaches its tensors through the runtime's operations only (see Part.chain_safe)
         self.chain_safe = all(getattr(part, "chain_safe", False)
@@ -165,5 +183,8 @@ class Block:
         if s.ffn_scale_name is not None and self.ffn is not None:
             self.ffn_scale = get(s.ffn_scale_name)
 
-    def forward(self, h, ctx, cache=None, write=True):
+    def forward(self, h, ctx, cache=None, write=True, normed=None):
+        """``normed``: the mixer's norm of h, already made (blocks with ``takes_ready_norm``)."""
+        if normed is not None:
+            return self._run(self, h, ctx, cache, write, normed)
         return self._run(self, h, ctx, cache, write)

@@ -7,7 +7,7 @@ where a router output past the real experts stands for an expert that returns x.
 at load ([experts, 2 F, C] with the gate rows first, and [experts, C, F]), so the kernels address an expert by its
 number.
 
-Options of the spec change the rule: sigmoid scores instead of a softmax, no correction, weights that are the chosen
+Options of the spec change the rule: a group judged by the sum of its largest choice scores, a constant on every weight, sigmoid scores instead of a softmax, no correction, weights that are the chosen
 scores as they are, a weight that multiplies the expert's input (sum expert(w x)) instead of its result, and one more
 expert that every token passes, whose result is added to the sum, times sigmoid(W_sg x) (one number per token) where
 the spec says so; experts without a gate matrix, W_down act(W_up x), whose stack is then [experts, F, C]. The expert
@@ -26,6 +26,7 @@ from .mlp import ACTIVATIONS, project_activated
 class RoutedExperts(FeedForward):
     chain_safe = True
     takes_out_dtype = True
+    takes_residual_scale = True
 
     @classmethod
     def kernels(cls, spec):
@@ -55,9 +56,13 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"unknown activation {self.activation!r} of {'gated' if self.gated else 'ungated'} experts")
         self.has_correction = bool(getattr(s, "correction", True))
         self.renormalize = bool(getattr(s, "renormalize", True))
+        self.group_best = int(getattr(s, "group_best", 1))
+        self.weight_scale = float(getattr(s, "weight_scale", 1.0))
+        if self.group_best < 1:
+            raise ValueError("a group's score is the sum of at least one choice score")
         # the plain rule keeps the call it always made; anything else names its options
         self.plain_rule = (self.scoring == "softmax" and self.has_correction and self.renormalize and not self.weight_input
-                           and self.shared_size is None)
+                           and self.shared_size is None and self.group_best == 1 and self.weight_scale == 1.0)
         self.w_router = self.correction = self.w_gate_up = self.w_down = None
         self.w_shared_gate_up = self.w_shared_down = None
 
@@ -107,7 +112,8 @@ class RoutedExperts(FeedForward):
         if self.plain_rule:
             return (*ops.moe_route(x, self.w_router, self.correction, s.groups, s.keep_groups, s.top), None)
         routed = ops.moe_route(x, self.w_router, self.correction, s.groups, s.keep_groups, s.top, scoring=self.scoring,
-                               renormalize=self.renormalize, extra=int(self.shared_gate))
+                               renormalize=self.renormalize, extra=int(self.shared_gate), group_best=self.group_best,
+                               weight_scale=self.weight_scale)
         return routed if self.shared_gate else (*routed, None)
 
     def _experts(self, x, update=None):
@@ -134,10 +140,9 @@ class RoutedExperts(FeedForward):
         return self._experts(x, update=(h, a, scale_a, scale_b, mult))
 
     def forward(self, x, ctx, residual=None, out_dtype=None):
-        ops = self.rt.ops
+        if residual is not None:  # added by the experts' last kernel
+            return self._experts(x, update=(residual, None, None, None, self.residual_scale))
         out = self._experts(x)  # float32 [N, C]
-        if residual is not None:
-            return ops.scaled_add(residual, out, None, None, None, 1.0)
         return out if out_dtype in (None, torch.float32) else out.to(out_dtype)
 
 

@@ -1,5 +1,5 @@
 """Mixers whose cache is a matrix state per head: gated linear attention, linear attention with a constant decay per
-head, and the gated delta rule.
+head, linear attention whose forget gate also writes, and the gated delta rule.
 
 All keep, per request and head, a float32 matrix S [key_dim, value_dim] in the request's state slot, update it
 token by token and read it out with the token's query, so a step of any length continues from what earlier
@@ -11,6 +11,9 @@ steps left and a request's cost per token does not grow with its length.
 * ``DecayedLinearAttention``: S <- decay_h S + k_t v_t^T, o_t = S^T q_t with one constant decay per head (the
   recurrence of Qin et al.'s "Lightning Attention-2" without its chunking); q, k and v pass silu, the read-out of all
   heads is normed as one row, gated by sigmoid(W_g x) and projected.
+* ``HGRN2``: S <- diag(f_t) S + (1 - f_t) v_t^T, o_t = S^T q_t with a forget gate per key channel, f = l + (1 - l)
+  sigmoid(W_f x + b), that stands in for the key; q passes silu. (Qin et al., "HGRN2: Gated Linear RNNs with State
+  Expansion", state the recurrence.)
 * ``GatedDelta``: S <- g_t S; u = beta_t (v_t - S^T k_t); S <- S + k_t u^T; o_t = S^T q_t, after a short causal
   convolution and silu on q, k and v and unit-length q and k. The convolution's last inputs are part of the state.
 
@@ -151,6 +154,61 @@ class DecayedLinearAttention(Mixer):
         return project(self.rt, y, self.w_out, out_dtype=out_dtype, residual=residual)
 
 
+class HGRN2(Mixer):
+    takes_normed = True
+    chain_safe = True
+    takes_out_dtype = True
+    takes_residual_scale = True
+
+    @classmethod
+    def kernels(cls, spec):
+        return ("recurrent",)
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        self.w_in = self.w_out = self.b_f = self.lower = self.norm = None
+
+    def _n(self, local):
+        return renamed(self.spec, local)
+
+    def params(self):
+        s = self.spec
+        c, hd, hv = s.hidden_size, s.num_heads * s.key_dim, s.num_heads * s.value_dim
+        return {
+            self._n("q"): Param((hd, c)),
+            self._n("f"): Param((hd, c)),
+            self._n("f.b"): Param((hd,), role="vector", mean=2.0),
+            self._n("lower"): Param((hd,), role="vector", mean=0.5),
+            self._n("v"): Param((hv, c)),
+            self._n("norm"): Param((s.value_dim,), role="vector", mean=1.0),
+            self._n("o"): Param((c, hv)),
+        }
+
+    def load(self, get):
+        self.w_in = stack_rows([get(self._n(n)) for n in ("q", "f", "v")])
+        self.b_f, self.lower, self.norm = get(self._n("f.b")), get(self._n("lower")), get(self._n("norm"))
+        self.w_out = get(self._n("o"))
+
+    def cache(self):
+        s = self.spec
+        return StateSpec((s.num_heads, s.value_dim, s.key_dim), torch.float32)  # S transposed, as the scan kernels keep it
+
+    def core(self, proj, ctx, cache, write=True, out=None, out_scale=1.0):
+        """From the input product ``proj`` [N, rows of w_in] to what the output product reads, times ``out_scale``."""
+        s, ops = self.spec, self.rt.ops
+        hd, hv = s.num_heads * s.key_dim, s.num_heads * s.value_dim
+        o = ops.hgrn2_scan(proj[:, :hd], proj[:, hd : 2 * hd], proj[:, 2 * hd : 2 * hd + hv], self.b_f, self.lower, cache.state,
+                           ctx.cu_seqlens, ctx.slots, s.num_heads, s.key_dim, s.value_dim, write=write,
+                           longest=getattr(ctx, "max_query_len", None))
+        return ops.gated_rmsnorm(o, self.norm, s.norm_eps, None, s.num_heads, s.value_dim, self.rt.dtype, out=out, out_scale=out_scale)
+
+    def forward(self, x, ctx, cache=None, residual=None, write=True, out_dtype=None):
+        # the product leaves float32: the forget gates are computed from it, and the state is float32 as well
+        proj = project(self.rt, x, self.w_in, out_dtype=torch.float32)
+        y = self.core(proj, ctx, cache, write, out_scale=1.0 if residual is None else self.residual_scale)
+        return project(self.rt, y, self.w_out, out_dtype=out_dtype, residual=residual)
+
+
 class GatedDelta(Mixer):
     takes_normed = True
     chain_safe = True
@@ -224,4 +282,5 @@ class GatedDelta(Mixer):
 
 register_mixer("gated_linear_attention", GatedLinearAttention)
 register_mixer("gated_delta", GatedDelta)
+register_mixer("hgrn2", HGRN2)
 register_mixer("decayed_linear_attention", DecayedLinearAttention)
