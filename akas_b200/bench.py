@@ -69,6 +69,8 @@ def prefill_flops(runner: ModelRunner, tokens: int, start: int = 0) -> float:
             # (query, key, head, channel) for each of the two products
             if spec.window:
                 pairs = sum(min(start + i + 1, spec.window + getattr(spec, "keep_first", 0)) for i in range(tokens))
+                if getattr(spec, "pool", None):  # and the blocks in front of the window
+                    pairs += sum(max(0, start + i - spec.window + 1) // spec.pool for i in range(tokens))
             else:
                 pairs = tokens * start + tokens * (tokens + 1) / 2
             flops += 2.0 * pairs * spec.num_heads * (spec.head_dim + getattr(spec, "value_dim", spec.head_dim))
@@ -76,7 +78,7 @@ def prefill_flops(runner: ModelRunner, tokens: int, start: int = 0) -> float:
             # as computed: every head's query against the cached rows [latent, rotated part], weights times the latent
             pairs = sum(min(start + i + 1, spec.window) for i in range(tokens)) if spec.window else tokens * start + tokens * (tokens + 1) / 2
             flops += 2.0 * pairs * spec.num_heads * (2 * spec.kv_rank + spec.rope_dim)
-        elif kind in ("gated_linear_attention", "gated_delta", "decayed_linear_attention"):
+        elif kind in ("gated_linear_attention", "gated_delta", "decayed_linear_attention", "hgrn2"):
             # the matrix state: decay and rank-one update, read-out (and the delta rule's read before the update)
             per = 6.0 if kind == "gated_delta" else 4.0
             flops += per * tokens * spec.num_heads * spec.key_dim * spec.value_dim
@@ -90,6 +92,8 @@ def decode_bytes(runner: ModelRunner, contexts: Sequence[int]) -> float:
     total = float(runner.weight_bytes)
     if runner.model.head is not runner.model.embedding:
         total -= runner.model.embedding.numel() * elem  # an untied embedding is only gathered from
+    if runner.model.bigram is not None:
+        total -= runner.model.bigram.numel() * elem
     views = []
     for view in runner.cache.views:
         views.extend(view if isinstance(view, tuple) else [view])
@@ -102,6 +106,9 @@ def decode_bytes(runner: ModelRunner, contexts: Sequence[int]) -> float:
                 per_token = spec.width * elem
             else:
                 per_token = spec.num_kv_heads * (spec.head_dim + (getattr(spec, "v_head_dim", None) or spec.head_dim)) * elem
+            if hasattr(spec, "block"):  # one key and one value per block of tokens, wherever the layer's window begins
+                total += sum(per_token * (c // spec.block) for c in contexts)
+                continue
             for c in contexts:
                 total += per_token * (min(c, spec.window + getattr(spec, "keep_first", 0)) if spec.window else c)
         else:
@@ -545,6 +552,26 @@ def pekodra_shape_config(name: str) -> dict:
                 layers=[dict(type="attention", mixer=attention, mlp=moe if i % 2 else dense) for i in range(runs - 2)])
 
 
+# Nuzulorn at LFM2's layer sizes: the same width, vocabulary and number of layers. The mixers take turns: attention with
+# LFM2's head counts inside a window of 1,024 with blocks of 16 tokens in front of it, a matrix state with forget gates (a
+# head per 128 channels of the width, keys of 64 and values of 128, like Gigusun's gated linear attention), and capped
+# attention with LFM2's head counts over the whole context. Every layer has 16 experts in 4 groups of which 2 stay, 4 per
+# token, each a quarter as wide as LFM2's feed-forward: as Girelix's 14 experts and 2 identities.
+def nuzulorn_shape_config(name: str) -> dict:
+    lfm2 = config_from_shape(name)
+    c, ff3 = lfm2.hidden_size, lfm2.feed_forward_size
+    heads = dict(heads=lfm2.num_attention_heads, kv_heads=lfm2.num_key_value_heads, dim=lfm2.head_dim, vdim=lfm2.head_dim,
+                 scale=lfm2.head_dim ** -0.5)
+    window = dict(heads, mask=dict(size=1024, pool=16), rot=dict(base=500000.0, dims=lfm2.head_dim))
+    capped = dict(heads, softcap=30.0, q_temp=dict(coef=0.3, every=512))
+    gates = dict(heads=c // 128, dim=64, vdim=128)
+    mlp = dict(kind="moe", expert=dict(ff=ff3 // 4), router=dict(experts=16, top=4, groups=dict(count=4, keep=2), scale=1.5))
+    mixers = (("attention", window), ("hgrn2", gates), ("attention_2", capped))
+    return dict(architecture="Nuzulorn", width=c, vocab=lfm2.vocab_size, norm=dict(eps=1e-5), residual_mult=0.5,
+                embedding=dict(bigram=dict(buckets=lfm2.vocab_size, mul_prev=31337, mul_cur=97)),
+                layers=[dict(type=mixers[i % 3][0], mixer=mixers[i % 3][1], mlp=mlp) for i in range(len(lfm2.layer_kinds))])
+
+
 def config_from_shape(name: str):
     from .config import config_from_dict
 
@@ -571,7 +598,7 @@ def compare_designs(shape: str = "1.2b", prompt: int = 2048, batches=(8, 64), st
 
     rows = []
     shapes = {"lfm2": shape_config, "gigusun": gigusun_shape_config, "girelix": girelix_shape_config,
-              "penopel": penopel_shape_config, "kidarax": kidarax_shape_config, "pekodra": pekodra_shape_config}
+              "penopel": penopel_shape_config, "kidarax": kidarax_shape_config, "pekodra": pekodra_shape_config, "nuzulorn": nuzulorn_shape_config}
     for design, data in ((name, shapes[name](shape)) for name in designs):
         say(f"{design} {shape}: writing random weights")
         model_config = config_from_dict(data)

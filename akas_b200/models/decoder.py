@@ -121,8 +121,10 @@ class Decoder:
         # adds in place into the rows [e + 1], which the average in front of it has written, and so leaves its result there.
         history = None
         if self.averages:
-            history = torch.empty((len(self.schedule) + 1, ctx.num_tokens, spec.hidden_size), dtype=torch.float32,
-                                  device=self.embedding.device)
+            words = ctx.num_tokens * spec.hidden_size
+            pitch = -(-words // 64) * 64  # every entry's rows start on 256 bytes, as rows of their own would
+            history = torch.empty((len(self.schedule) + 1, pitch), dtype=torch.float32, device=self.embedding.device)
+            history = history[:, :words].view(-1, ctx.num_tokens, spec.hidden_size)
         started = False  # whether the embedding's output lies in the first two rows of the buffer already
         if spec.bigram is not None:
             b = spec.bigram

@@ -465,9 +465,9 @@ def bigram_embedding(token_ids, table, pairs, mul_prev, mul_cur, state, cu_seqle
     if out is None:
         first, both = torch.empty((n, c), dtype=torch.float32, device=table.device), None
     else:
-        if out.dtype != torch.float32 or out.shape != (2, n, c) or not out.is_contiguous():
-            raise ValueError("bigram_embedding writes to dense float32 [2, N, C]")
         first, both = out[0], out[1]
+        if out.dtype != torch.float32 or out.shape != (2, n, c) or not first.is_contiguous():
+            raise ValueError("bigram_embedding writes to float32 [2, N, C] whose halves are dense")
     _check(_fn("elementwise", "akas_bigram_embedding")(
         _ptr(token_ids), _ptr(_dense(table, "table")), _ptr(_dense(pairs, "pairs")), int(mul_prev), int(mul_cur), pairs.shape[0] - 1,
         _ptr(state), _ptr(cu_seqlens), _ptr(seq_of_token), _ptr(slots), _ptr(first), _ptr(both), n, c, _code(table), _stream()),
@@ -477,18 +477,18 @@ def bigram_embedding(token_ids, table, pairs, mul_prev, mul_cur, state, cu_seqle
 
 @_flushes
 def depth_average(history, count, weights, out, rows=None, norm=None):
-    """sum_j weights[j] * history[j] over j < count for dense float32 history [.., N, C] (``rows``: of those rows alone).
+    """sum_j weights[j] * history[j] over j < count for float32 history [.., N, C] of dense [N, C] (``rows``: of those rows alone).
     ``norm`` = (weight, eps, zero_centered, dtype): where the product behind that RMSNorm would not compute it on its way
     in, the same pass makes it. Returns (result, normed result or None)."""
     _, n, c = history.shape
-    if history.dtype != torch.float32 or not history.is_contiguous() or weights.dtype != torch.float32 or weights.numel() != count:
-        raise ValueError("depth_average takes dense float32 history [.., N, C] and one float32 weight per summand")
+    if history.dtype != torch.float32 or not history[0].is_contiguous() or weights.dtype != torch.float32 or weights.numel() != count:
+        raise ValueError("depth_average takes float32 history [.., N, C] of dense [N, C] and one float32 weight per summand")
     m = rows.numel() if rows is not None else n
     if out is None:
         out = torch.empty((m, c), dtype=torch.float32, device=history.device)
     elif out.dtype != torch.float32 or out.shape != (m, c) or not out.is_contiguous():
         raise ValueError("depth_average writes to dense float32 rows")
-    args = (_ptr(history), n * c, count, _ptr(weights), _ptr(out), _ptr(rows), m, c)
+    args = (_ptr(history), history.stride(0), count, _ptr(weights), _ptr(out), _ptr(rows), m, c)
     if norm is not None:
         weight, eps, zero_centered, dtype = norm
         if dtype == torch.float32 or not (decode_products == "stream" or _skinny_fits(m, c)):

@@ -157,3 +157,29 @@ def test_generate_runs_a_pekodra_folder(tmp_path, capsys):
     for extra in ([], ["--temperature", "0.7", "--top-k", "20", "--seed", "2", "--dtype", "float32"]):
         main(["generate", "--model", str(tmp_path / "k"), "--prompt", "5 17 3 9", "--max-tokens", "7", "--ignore-eos", *extra])
         assert len(capsys.readouterr().out.split()) == 7
+
+
+def test_random_and_inspect_take_a_nuzulorn_configuration(tmp_path, capsys):
+    import tiny_nuzulorn
+
+    config = tiny_nuzulorn.CONFIGS["mix"]
+    main(["random", "--out", str(tmp_path / "k"), "--config", json.dumps(config), "--seed", "4"])
+    capsys.readouterr()
+    main(["inspect", "--model", str(tmp_path / "k")])
+    report = json.loads(capsys.readouterr().out)
+    assert report["architecture"] == "Nuzulorn" and report["config"] == json.loads(json.dumps(config))
+    assert {"embed", "bigram", "l0.norm1", "l0.norm2", "l0.mix.o.b", "l0.mix.g", "l0.mlp.correction", "l0.mlp.e5.gate", "l0.dwa", "l1.mix.lower",
+            "l1.mix.f.b", "l1.mix.norm", "l2.mix.sink", "l4.dwa", "final.norm"} <= set(report["inventory"])
+    # no head of its own, no output bias or gate of a capped layer, no bias of the matrix state's other projections
+    assert not {"head", "l2.mix.o.b", "l2.mix.g", "l1.mix.q.b", "l2.mlp.router"} & set(report["inventory"])
+
+
+@pytest.mark.gpu
+def test_generate_runs_a_nuzulorn_folder(tmp_path, capsys):
+    import tiny_nuzulorn
+
+    main(["random", "--out", str(tmp_path / "k"), "--config", json.dumps(tiny_nuzulorn.CONFIGS["mix"]), "--seed", "4"])
+    capsys.readouterr()
+    for extra in ([], ["--temperature", "0.7", "--top-k", "20", "--seed", "2", "--dtype", "float32"]):
+        main(["generate", "--model", str(tmp_path / "k"), "--prompt", "5 17 3 9", "--max-tokens", "7", "--ignore-eos", *extra])
+        assert len(capsys.readouterr().out.split()) == 7
