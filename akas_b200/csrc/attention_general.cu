@@ -247,6 +247,68 @@ pool_blocks_kernel(const T* __restrict__ k_pool, const T* __restrict__ v_pool, T
   }
 }
 
+// The same for head sizes that are multiples of 8, everything on 16 bytes: a thread owns 8 neighbouring channels of a
+// head's key or value and asks for up to 16 of the block's rows before it adds the first. A grid block looks at kPoolTokens
+// neighbouring tokens, so that a step of many tokens is not a launch of as many blocks most of which end at once.
+constexpr int kPoolTokens = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(64)
+pool_blocks8_kernel(const T* __restrict__ k_pool, const T* __restrict__ v_pool, T* __restrict__ k_blocks, T* __restrict__ v_blocks,
+                    const int* __restrict__ token_table, int token_width, const int* __restrict__ block_table, int block_width,
+                    const int* __restrict__ seq_of_token, const int* __restrict__ positions, int page_size, int block_page,
+                    int entries, int block, int G, int D, int V, int N) {
+  constexpr int ROWS = sizeof(T) == 2 ? 16 : 8;  // rows in flight
+  __shared__ int last[kPoolTokens], owner[kPoolTokens];
+  if (threadIdx.x < kPoolTokens) {
+    const int n = blockIdx.x * kPoolTokens + threadIdx.x;
+    const int req = n < N ? seq_of_token[n] : -1;
+    const int pos = n < N ? positions[n] : 0;
+    last[threadIdx.x] = pos;
+    owner[threadIdx.x] = (pos + 1) % block == 0 ? req : -1;
+  }
+  __syncthreads();
+  const int per = (D + V) / 8;
+  const int i = blockIdx.y * blockDim.x + threadIdx.x;
+  if (i >= G * per) return;
+  const int g = i / per, e = i % per * 8;
+  const bool key = e < D;
+  const T* src = key ? k_pool + e : v_pool + (e - D);
+  const int size = key ? D : V;
+  const float inv = 1.f / (float)block;
+  for (int u = 0; u < kPoolTokens; ++u) {
+    const int req = owner[u], pos = last[u];
+    if (req < 0) continue;
+    const int* table = token_table + (size_t)req * token_width;
+    const int page = block_table[(size_t)req * block_width + pos / block_page];
+    float sum[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    for (int t0 = pos - block + 1; t0 <= pos; t0 += ROWS) {
+      uint4 raw[ROWS][sizeof(T) / 2];
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r) {
+        const int t = min(t0 + r, pos);
+        const long long row = ((long long)table[t / page_size] * G + g) * page_size + t % page_size;
+#pragma unroll
+        for (int h = 0; h < (int)sizeof(T) / 2; ++h) raw[r][h] = reinterpret_cast<const uint4*>(src + row * size)[h];
+      }
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r) {
+        if (t0 + r <= pos) {
+          float x[8];
+          load8(reinterpret_cast<const T*>(&raw[r][0]), x);
+#pragma unroll
+          for (int c = 0; c < 8; ++c) sum[c] += x[c];
+        }
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < 8; ++c) sum[c] *= inv;
+    const long long row = ((long long)page * G + g) * entries + pos / block - (pos / block_page * block_page) / block;
+    if (key) store8(k_blocks + row * D + e, sum);
+    else store8(v_blocks + row * V + (e - D), sum);
+  }
+}
+
 // The blocks that a layer sees in front of its window (block 0: none): their pages, the block table with its width, the
 // tokens and the entries of a page, and the tokens of a block.
 template <typename T>
@@ -549,7 +611,18 @@ AKAS_API int akas_pool_blocks(const void* k_pool, const void* v_pool, void* k_bl
   if (N <= 0) return 0;
   if (block <= 0 || block_page <= 0 || page_size <= 0) return (int)cudaErrorInvalidValue;
   const int entries = (block_page + block - 1) / block;
-  const dim3 grid(N, N <= 64 ? max(1, min(16, (G * (D + V) + 127) / 128)) : 1);
+  const uintptr_t bases = (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)k_blocks | (uintptr_t)v_blocks;
+  if (D % 8 == 0 && V % 8 == 0 && bases % 16 == 0) {
+    const dim3 grid8((N + kPoolTokens - 1) / kPoolTokens, (G * ((D + V) / 8) + 63) / 64);
+#define AKAS_POOL8(T)                                                                                                          \
+  return launch_ordinary(pool_blocks8_kernel<T>, grid8, dim3(64), 0, stream, (const T*)k_pool, (const T*)v_pool, (T*)k_blocks, \
+                         (T*)v_blocks, token_table, token_width, block_table, block_width, seq_of_token, positions, page_size, \
+                         block_page, entries, block, G, D, V, N)
+    if (dtype == AKAS_F32) AKAS_POOL8(float);
+    AKAS_POOL8(bf16);
+#undef AKAS_POOL8
+  }
+  const dim3 grid(N, max(1, min(16, (G * (D + V) + 127) / 128)));
   if (dtype == AKAS_F32)
     return launch_ordinary(pool_blocks_kernel<float>, grid, dim3(128), 0, stream, (const float*)k_pool, (const float*)v_pool,
                            (float*)k_blocks, (float*)v_blocks, token_table, token_width, block_table, block_width, seq_of_token,

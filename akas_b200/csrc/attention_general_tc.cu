@@ -13,8 +13,10 @@
 // whose pitch is the caller's.
 //
 // Packed launches serve steps of single tokens (decoding): a block's rows are then the query heads that share one
-// key/value head, all at the token's position, so its keys and values are read once for the whole group; warps
-// without a live row only help with the copies. A packed launch may cut every request's key tiles into `splits`
+// key/value head, all at the token's position, so its keys and values are read once for the whole group. Up to 16 such
+// heads (general_decode_kernel) the four warps share them and take 16 keys of every tile each, with maxima and sums of
+// their own that meet in shared memory at the end; with more, a warp's rows are its own and warps without a live row
+// only help with the copies. A packed launch may cut every request's key tiles into `splits`
 // parts (gridDim.z): a block then walks its part only and leaves its unnormalised sums, its maximum and its sum of
 // weights in a scratch buffer, and general_merge_kernel adds the parts (and the sink's term, once) in the order of
 // their numbers: a decode step of a few requests with thousands of keys each fills the GPU that way.
@@ -377,6 +379,242 @@ general_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_po
   }
 }
 
+// The packed launch for groups of at most 16 heads: grid (key/value heads, requests, parts of the keys). All four warps
+// hold the same 16 query rows; warp w computes the scores of keys 16 w .. 16 w + 15 of every tile and adds their values.
+// Where a tile's rows lie is found two tiles ahead, one thread a row, and left in shared memory for the copies.
+template <int DKP, int DVP>
+__global__ void __launch_bounds__(WARPS * 32)
+general_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool, const bf16* __restrict__ v_pool,
+                      const int* __restrict__ block_table, int max_blocks, const int* __restrict__ cu_seqlens,
+                      const int* __restrict__ positions, bf16* __restrict__ out, Options opt, int page_size, int H, int KH, int D, int V,
+                      float* __restrict__ partial, int splits) {
+  constexpr int KSTRIDE = DKP + 8, VSTRIDE = DVP + 8;
+  constexpr int KCH = DKP / 8, VCH = DVP / 8, KS = DKP / 16, NB = DVP / 8;
+  static_assert(BK == WARPS * 16, "a warp takes 16 keys of a tile");
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  bf16* k_s = reinterpret_cast<bf16*>(smem_raw);  // [2][BK][KSTRIDE]; stage 0 first holds Q
+  bf16* v_s = k_s + 2 * BK * KSTRIDE;             // [2][BK][VSTRIDE]; at the end the warps' sums [WARPS][16][DVP] float32
+  __shared__ long long row_at[3][BK];             // a tile's rows in their pool (blocks of tokens: in theirs), -1: none
+  __shared__ float top_s[WARPS][16], sum_s[WARPS][16];
+
+  const int kvh = blockIdx.x, r = blockIdx.y;
+  const int q0 = cu_seqlens[r];
+  if (cu_seqlens[r + 1] <= q0) return;  // padding
+  const int group = H / KH;
+  const int pos = positions[q0];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int g = lane >> 2, t = lane & 3;
+  const int window = opt.window, keep = opt.window > 0 ? opt.keep_first : 0;
+  const int first_key = window > 0 ? max(0, pos - window + 1) : 0;
+  const int kt0 = first_key / BK, kt1 = pos / BK;
+  const int kept_tiles = min((keep + BK - 1) / BK, kt0);
+  const int blocks = opt.block > 0 ? first_key / opt.block : 0;  // blocks of tokens in front of the window
+  const int block_tiles = (blocks + BK - 1) / BK;
+  const int total = block_tiles + kept_tiles + (kt1 - kt0 + 1);
+  int i_begin = 0, i_end = total;
+  if (splits > 1) {
+    const int per = (total + splits - 1) / splits;
+    i_begin = min(total, (int)blockIdx.z * per);
+    i_end = min(total, i_begin + per);
+  }
+  auto tile_of = [&](int i) {
+    if (i < block_tiles) return -1 - i;
+    i -= block_tiles;
+    return i < kept_tiles ? i : kt0 + (i - kept_tiles);
+  };
+  auto find_row = [&](int i, int row) {  // where row `row` of the i-th tile lies
+    const int kt = tile_of(i);
+    long long at = -1;
+    if (kt < 0) {
+      const int b = (-1 - kt) * BK + row;
+      if (b < blocks) {
+        const int in = (b * opt.block + opt.block - 1) / opt.bpage;  // the page of the block's last token
+        const int page = opt.btable[(size_t)r * opt.bwidth + in];
+        if (page >= 0) at = ((long long)page * KH + kvh) * opt.entries + b - in * opt.bpage / opt.block;
+      }
+    } else {
+      const int key = kt * BK + row;
+      if (key <= pos && (key >= first_key || key < keep)) {
+        const int page = block_table[(size_t)r * max_blocks + key / page_size];
+        if (page >= 0) at = ((long long)page * KH + kvh) * page_size + key % page_size;
+      }
+    }
+    row_at[i % 3][row] = at;
+  };
+
+  for (int c = tid; c < 16 * KCH; c += WARPS * 32) {
+    const int row = c / KCH, col = (c % KCH) * 8;
+    const bf16* src = q + ((size_t)q0 * H + kvh * group + min(row, group - 1)) * D + min(col, D - 8);
+    cp_async16(k_s + row * KSTRIDE + col, src, row < group && col < D ? 16 : 0);
+  }
+  cp_async_commit();
+  if (i_begin + (tid >> 6) < i_end) find_row(i_begin + (tid >> 6), tid & 63);
+  cp_async_wait<0>();
+  __syncthreads();
+  uint32_t qf[KS][4];
+#pragma unroll
+  for (int ks = 0; ks < KS; ++ks) ldmatrix_x4(qf[ks], k_s + (lane & 15) * KSTRIDE + ks * 16 + (lane >> 4) * 8);
+  __syncthreads();
+
+  auto load_tile = [&](int i, int stage) {
+    const bool pooled = tile_of(i) < 0;
+    const bf16* kp = pooled ? opt.k_blocks : k_pool;
+    const bf16* vp = pooled ? opt.v_blocks : v_pool;
+    const long long pitch = pooled ? V : opt.vpitch;
+    bf16* ks_ = k_s + stage * BK * KSTRIDE;
+    bf16* vs_ = v_s + stage * BK * VSTRIDE;
+#pragma unroll 4
+    for (int c = tid; c < BK * (KCH + VCH); c += WARPS * 32) {
+      const int row = c / (KCH + VCH), ch = c % (KCH + VCH);
+      const long long at = row_at[i % 3][row];
+      const long long base = at >= 0 ? at : 0;
+      if (ch < KCH) {
+        const int col = ch * 8;
+        cp_async16(ks_ + row * KSTRIDE + col, kp + base * D + min(col, D - 8), at >= 0 && col < D ? 16 : 0);
+      } else {
+        const int col = (ch - KCH) * 8;
+        cp_async16(vs_ + row * VSTRIDE + col, vp + base * pitch + min(col, V - 8), at >= 0 && col < V ? 16 : 0);
+      }
+    }
+    cp_async_commit();
+  };
+
+  float o[NB][4];
+#pragma unroll
+  for (int nb = 0; nb < NB; ++nb) { o[nb][0] = o[nb][1] = o[nb][2] = o[nb][3] = 0.f; }
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  const int head2[2] = {kvh * group + min(g, group - 1), kvh * group + min(g + 8, group - 1)};
+  const bool biased = opt.r1 != nullptr, linear = biased && opt.r2 == nullptr;
+  const float unit = linear ? kLog2e : 1.f;  // (r1 ln(1 + r2 d) in units of log2 e is r1 lg2(1 + r2 d))
+  const float r1[2] = {biased ? unit * opt.r1[head2[0]] : 0.f, biased ? unit * opt.r1[head2[1]] : 0.f};
+  const float r2[2] = {biased && !linear ? opt.r2[head2[0]] : 0.f, biased && !linear ? opt.r2[head2[1]] : 0.f};
+  const float cap2 = opt.cap * kLog2e, scale2 = opt.scale * kLog2e, scale_cap = opt.cap > 0.f ? opt.scale / opt.cap : 0.f;
+
+  if (i_begin < i_end) load_tile(i_begin, 0);
+  for (int i = i_begin; i < i_end; ++i) {
+    const int kt = tile_of(i);
+    const int stage = (i - i_begin) & 1;
+    if (i + 1 < i_end) {
+      load_tile(i + 1, stage ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const bf16* ks_ = k_s + stage * BK * KSTRIDE + warp * 16 * KSTRIDE;
+    const bf16* vs_ = v_s + stage * BK * VSTRIDE + warp * 16 * VSTRIDE;
+    float s[2][4] = {};
+#pragma unroll
+    for (int ks = 0; ks < KS; ++ks) {
+      uint32_t b[4];
+      ldmatrix_x4(b, ks_ + ((lane & 7) + (lane >> 4) * 8) * KSTRIDE + ks * 16 + ((lane >> 3) & 1) * 8);
+      mma_bf16(s[0], qf[ks], b[0], b[1]);
+      mma_bf16(s[1], qf[ks], b[2], b[3]);
+    }
+    float m_new[2] = {m_run[0], m_run[1]};
+#pragma unroll
+    for (int nb = 0; nb < 2; ++nb) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int row = warp * 16 + nb * 8 + 2 * t + (e & 1);
+        const int key = kt * BK + row, dist = pos - key;
+        const bool seen = kt < 0 ? (-1 - kt) * BK + row < blocks
+                                 : dist >= 0 && (window <= 0 || dist < window || key < keep);
+        float x = opt.cap > 0.f ? cap2 * fast_tanh(s[nb][e] * scale_cap) : s[nb][e] * scale2;
+        if (linear) x = fmaf(-r1[e >> 1], (float)dist, x);
+        else if (biased) x -= r1[e >> 1] * fast_log2(fmaf(r2[e >> 1], (float)max(dist, 0), 1.f));
+        s[nb][e] = seen ? x : -INFINITY;
+        m_new[e >> 1] = fmaxf(m_new[e >> 1], s[nb][e]);
+      }
+    }
+    float corr[2], m_use[2];
+#pragma unroll
+    for (int h2 = 0; h2 < 2; ++h2) {
+      m_new[h2] = fmaxf(m_new[h2], __shfl_xor_sync(0xffffffffu, m_new[h2], 1));
+      m_new[h2] = fmaxf(m_new[h2], __shfl_xor_sync(0xffffffffu, m_new[h2], 2));
+      m_use[h2] = m_new[h2] == -INFINITY ? 0.f : m_new[h2];
+      corr[h2] = fast_exp2(m_run[h2] - m_use[h2]);
+      m_run[h2] = m_new[h2];
+    }
+    uint32_t pf[4];
+    float l_add[2] = {0.f, 0.f};
+#pragma unroll
+    for (int nb = 0; nb < 2; ++nb) {
+      const float p0 = fast_exp2(s[nb][0] - m_use[0]), p1 = fast_exp2(s[nb][1] - m_use[0]);
+      const float p2 = fast_exp2(s[nb][2] - m_use[1]), p3 = fast_exp2(s[nb][3] - m_use[1]);
+      l_add[0] += p0 + p1;
+      l_add[1] += p2 + p3;
+      pf[nb * 2] = pack_bf16(p0, p1);
+      pf[nb * 2 + 1] = pack_bf16(p2, p3);
+    }
+#pragma unroll
+    for (int h2 = 0; h2 < 2; ++h2) l_run[h2] = l_run[h2] * corr[h2] + l_add[h2];
+#pragma unroll
+    for (int nb = 0; nb < NB; ++nb) {
+      o[nb][0] *= corr[0]; o[nb][1] *= corr[0];
+      o[nb][2] *= corr[1]; o[nb][3] *= corr[1];
+    }
+#pragma unroll
+    for (int np = 0; np < NB / 2; ++np) {
+      uint32_t b[4];
+      ldmatrix_x4_trans(b, vs_ + ((lane & 7) + ((lane >> 3) & 1) * 8) * VSTRIDE + np * 16 + (lane >> 4) * 8);
+      mma_bf16(o[2 * np], pf, b[0], b[1]);
+      mma_bf16(o[2 * np + 1], pf, b[2], b[3]);
+    }
+    if (tid < BK && i + 2 < i_end) find_row(i + 2, tid);
+    __syncthreads();
+  }
+
+#pragma unroll
+  for (int h2 = 0; h2 < 2; ++h2) {
+    l_run[h2] += __shfl_xor_sync(0xffffffffu, l_run[h2], 1);
+    l_run[h2] += __shfl_xor_sync(0xffffffffu, l_run[h2], 2);
+    if (t == 0) {
+      top_s[warp][g + 8 * h2] = m_run[h2];
+      sum_s[warp][g + 8 * h2] = l_run[h2];
+    }
+  }
+  float* sums = reinterpret_cast<float*>(v_s);
+#pragma unroll
+  for (int nb = 0; nb < NB; ++nb) {
+    float* dst = sums + (warp * 16 + g) * DVP + nb * 8 + 2 * t;
+    dst[0] = o[nb][0];
+    dst[1] = o[nb][1];
+    dst[8 * DVP] = o[nb][2];
+    dst[8 * DVP + 1] = o[nb][3];
+  }
+  __syncthreads();
+  const bool sunk = splits <= 1 && (opt.sink || opt.sinks != nullptr);  // with parts, the merge adds the sink's term
+  const bool by_channel = opt.gate != nullptr && opt.gate_channels;
+  for (int c = tid; c < group * V; c += WARPS * 32) {
+    const int row = c / V, ch = c % V, head = kvh * group + row;
+    const float sink2 = opt.sinks != nullptr ? opt.sinks[head] * kLog2e : 0.f;
+    float top = sunk ? sink2 : -INFINITY;
+#pragma unroll
+    for (int w = 0; w < WARPS; ++w) top = fmaxf(top, top_s[w][row]);
+    float acc = 0.f, denom = sunk ? exp2f(sink2 - top) : 0.f;
+#pragma unroll
+    for (int w = 0; w < WARPS; ++w) {
+      const float f = top_s[w][row] == -INFINITY ? 0.f : exp2f(top_s[w][row] - top);
+      acc = fmaf(f, sums[(w * 16 + row) * DVP + ch], acc);
+      denom = fmaf(f, sum_s[w][row], denom);
+    }
+    if (splits > 1) {
+      float* dst = partial + (((size_t)q0 * H + head) * splits + blockIdx.z) * (V + 2);
+      dst[ch] = acc;
+      if (ch == 0) {
+        dst[V] = top;
+        dst[V + 1] = denom;
+      }
+      continue;
+    }
+    float inv = denom > 0.f ? opt.out_scale / denom : 0.f;
+    if (by_channel) inv *= gate_of(opt, (size_t)q0, head, V, ch);
+    else if (opt.gate != nullptr) inv *= gate_at(opt, (size_t)q0 * opt.ldg + head);
+    out[(size_t)q0 * opt.ldo + (size_t)head * V + ch] = __float2bfloat16_rn(acc * inv);
+  }
+}
+
 // One block per (request of one token, head): the parts' sums, rescaled to the common maximum (the sink's logit
 // included) and added in the order of the parts; then the division, the gate and the constant. The first warp reads
 // every part's maximum and weight sum at once (two parts a lane) and leaves a factor per part in shared memory.
@@ -443,9 +681,15 @@ int launch(const void* q, const void* k_pool, const void* v_pool, const int* blo
     const cudaError_t e = cudaFuncSetAttribute(general_prefill_kernel<DKP, DVP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                tiles_bytes + (kTableMost + kTableBefore + kTableAfter) * (int)sizeof(float));
     if (e != cudaSuccess) return (int)e;
+    const cudaError_t d = cudaFuncSetAttribute(general_decode_kernel<DKP, DVP>, cudaFuncAttributeMaxDynamicSharedMemorySize, tiles_bytes);
+    if (d != cudaSuccess) return (int)d;
     configured[device] = true;
   }
-  const int err = launch_ordinary(general_prefill_kernel<DKP, DVP>, dim3(packed ? KH : H, tiles, splits), dim3(WARPS * 32), (size_t)smem,
+  const int err = packed && H / KH <= 16
+      ? launch_ordinary(general_decode_kernel<DKP, DVP>, dim3(KH, R, splits), dim3(WARPS * 32), (size_t)tiles_bytes, stream, (const bf16*)q,
+                        (const bf16*)k_pool, (const bf16*)v_pool, block_table, max_blocks, cu_seqlens, positions, (bf16*)out, opt,
+                        page_size, H, KH, D, V, partial, splits)
+      : launch_ordinary(general_prefill_kernel<DKP, DVP>, dim3(packed ? KH : H, tiles, splits), dim3(WARPS * 32), (size_t)smem,
                                   stream, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, block_table, max_blocks,
                                   cu_seqlens, positions, (bf16*)out, opt, page_size, H, KH, D, V, R, packed, table, partial, splits);
   if (err || splits <= 1) return err;

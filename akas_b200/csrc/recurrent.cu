@@ -737,7 +737,8 @@ __device__ __forceinline__ float4 norm_weight4(const float* __restrict__ w, int 
   return w != nullptr ? *reinterpret_cast<const float4*>(w + j) : make_float4(1.f, 1.f, 1.f, 1.f);
 }
 
-template <typename TG, typename TO>
+// NI: a row of at most NI * 128 channels stays in registers (the fewer a row needs, the more warps an SM holds).
+template <typename TG, typename TO, int NI>
 __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps,
                                      const TG* __restrict__ gate, long long ldg, TO* __restrict__ out, int N, int H, int V,
                                      int sigmoid, float out_scale, long long ldo) {
@@ -752,11 +753,11 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const float* _
     // four channels a lane: 16-byte reads of o, 8- or 16-byte reads of the gate and writes of the result. A row of at
     // most 1,024 channels stays in registers between the sum and the result, with its weights and gates asked for in
     // the same trip to memory (a step of few tokens is a handful of warps that only wait).
-    if (V <= 1024) {
-      float4 x[8], wv[8];
-      float gv[8][4];
+    if (V <= NI * 128) {
+      float4 x[NI], wv[NI];
+      float gv[NI][4];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < NI; ++i) {
         const int j = lane * 4 + i * 128;
         if (j < V) {
           x[i] = *reinterpret_cast<const float4*>(row + j);
@@ -768,7 +769,7 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const float* _
       ss = warp_sum(ss);
       const float inv = out_scale / sqrtf(ss / (float)V + eps);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < NI; ++i) {
         const int j = lane * 4 + i * 128;
         if (j < V) {
 #pragma unroll
@@ -967,12 +968,14 @@ AKAS_API int akas_gated_rmsnorm(const float* o, const float* w, float eps, const
   if (N <= 0 || H <= 0) return 0;
   const long long items = (long long)N * H;
   const int blocks = (int)((items + 7) / 8);
-#define AKAS_GN(TG, TO) \
-  return launch_ordinary(gated_rmsnorm_kernel<TG, TO>, dim3(blocks), dim3(256), 0, stream, o, w, eps, (const TG*)gate, ldg, (TO*)out, N, H, V, \
+#define AKAS_GN_ROWS(TG, TO, NI) \
+  return launch_ordinary(gated_rmsnorm_kernel<TG, TO, NI>, dim3(blocks), dim3(256), 0, stream, o, w, eps, (const TG*)gate, ldg, (TO*)out, N, H, V, \
                          sigmoid, out_scale, ldo)
-  if (gate_dtype == AKAS_F32 && out_dtype == AKAS_F32) AKAS_GN(float, float);
-  if (gate_dtype == AKAS_F32) AKAS_GN(float, bf16);
-  if (out_dtype == AKAS_F32) AKAS_GN(bf16, float);
-  AKAS_GN(bf16, bf16);
+#define AKAS_GN(TG, TO) { if (V <= 128) AKAS_GN_ROWS(TG, TO, 1); if (V <= 256) AKAS_GN_ROWS(TG, TO, 2); AKAS_GN_ROWS(TG, TO, 8); }
+  if (gate_dtype == AKAS_F32 && out_dtype == AKAS_F32) AKAS_GN(float, float)
+  if (gate_dtype == AKAS_F32) AKAS_GN(float, bf16)
+  if (out_dtype == AKAS_F32) AKAS_GN(bf16, float)
+  AKAS_GN(bf16, bf16)
 #undef AKAS_GN
+#undef AKAS_GN_ROWS
 }

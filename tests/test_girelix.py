@@ -45,9 +45,10 @@ def compare(got, want, dtype, what):
         rows = np.arange(len(logits)) if dtype == "float32" else np.nonzero(held)[0]
         if dtype != "float32":
             # positions whose routing was clear are held one by one; over all positions, the typical error is held too
-            # (a choice that fell the other way is rare and moves one position far: the median does not see it)
+            # (a choice that fell the other way is rare and moves one position far: the median does not see it; of a few
+            # positions there is no typical error)
             error = np.abs(got[rid] - logits).max(axis=-1) / np.abs(logits).max()
-            assert np.median(error) <= 0.5 * TOL[dtype], f"{what}: request {rid}: median error {np.median(error):.3g}"
+            assert len(error) <= 3 or np.median(error) <= 0.5 * TOL[dtype], f"{what}: request {rid}: median error {np.median(error):.3g}"
             if len(rows) == 0:
                 continue
         bad = traces.first_bad(got[rid][rows], logits[rows], TOL[dtype])
